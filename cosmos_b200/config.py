@@ -104,7 +104,164 @@ def super_config(**kw) -> MoTConfig:
     return replace(base, **kw)
 
 
+# --------------------------------------------------------------------------- config-declared decoder stacks
+@dataclass(frozen=True)
+class AttentionSpec:
+    """Attention mixer of a stack layer. The optional mechanisms are switches, so that another design can combine them
+    differently: sliding window (None = unlimited), distance bias `r1 ln(1 + r2 (i - j))` per head, RMS norm of each
+    value head, mixing of the values with those of an earlier layer, q/k/v biases."""
+    heads: int
+    kv_heads: int
+    dim: int                      # query / key head size
+    vdim: int                     # value head size
+    scale: float
+    window: Optional[int] = None  # keys seen by a query, itself included
+    distance_bias: bool = False
+    value_norm: bool = False
+    value_mix: bool = False       # the first such layer gives its values, the others mix them in
+    qkv_bias: bool = False
+
+    @property
+    def qkv_cols(self) -> int:
+        return self.heads * self.dim + self.kv_heads * (self.dim + self.vdim)
+
+
+@dataclass(frozen=True)
+class MoESpec:
+    """Experts chosen by a table over token ids: table [vocab, top], each chosen expert with weight 1 / top; an expert is
+    down(gelu(up(h))) without biases (erf gelu)."""
+    experts: int
+    top: int
+    ff: int
+
+
+@dataclass(frozen=True)
+class StackLayerSpec:
+    mixer: AttentionSpec
+    mlp: Optional[MoESpec] = None
+
+
+@dataclass
+class StackConfig:
+    """A decoder whose layers are listed one by one (models/stack.py)."""
+    name: str
+    architecture: str
+    vocab_size: int
+    d_model: int
+    layers: Tuple[StackLayerSpec, ...]
+    embed_scale: float = 1.0
+    norm_eps: float = 1e-6
+    norm_groups: int = 1
+    init_std: float = 0.02
+
+    @property
+    def n_layers(self) -> int:
+        return len(self.layers)
+
+    @property
+    def rms_eps(self) -> float:
+        return self.norm_eps
+
+    def validate(self) -> "StackConfig":
+        if self.vocab_size < 1 or self.d_model < 1 or self.norm_groups < 1 or self.d_model % self.norm_groups:
+            raise ValueError("vocab and width must be positive and the width a multiple of the norm groups")
+        first = None
+        for i, layer in enumerate(self.layers):
+            m = layer.mixer
+            if min(m.heads, m.kv_heads, m.dim, m.vdim) < 1 or m.heads % m.kv_heads:
+                raise ValueError(f"layer {i}: heads must be a positive multiple of kv_heads")
+            if m.window is not None and m.window < 1:
+                raise ValueError(f"layer {i}: the window holds at least the token itself")
+            if m.value_mix:
+                if first is None:
+                    first = m
+                elif (m.kv_heads, m.vdim) != (first.kv_heads, first.vdim):
+                    raise ValueError(f"layer {i}: mixed values need the first mixing layer's kv_heads and vdim")
+            if layer.mlp is not None and not 1 <= layer.mlp.top <= layer.mlp.experts:
+                raise ValueError(f"layer {i}: top must be between 1 and the number of experts")
+        return self
+
+    def to_dict(self) -> Dict:
+        return ARCHITECTURES[self.architecture][1](self)
+
+
+def lederax_config_from_dict(doc: Dict, name: str = "Lederax") -> StackConfig:
+    """config.json of a Lederax model."""
+    layers = []
+    for i, entry in enumerate(doc["layers"]):
+        if entry["type"] != "attention":
+            raise ValueError(f"layer {i}: unknown mixer type {entry['type']!r}")
+        m = entry["mixer"]
+        mask = m.get("mask")
+        mixer = AttentionSpec(heads=int(m["heads"]), kv_heads=int(m["kv_heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]),
+                              scale=float(m["scale"]), window=int(mask["size"]) if mask else None, distance_bias=True,
+                              value_norm=True, value_mix=bool(m.get("v_mix", False)), qkv_bias=True)
+        mlp = entry.get("mlp")
+        if mlp is not None:
+            if mlp.get("kind") != "moe":
+                raise ValueError(f"layer {i}: unknown feed-forward kind {mlp.get('kind')!r}")
+            mlp = MoESpec(experts=int(mlp["router"]["experts"]), top=int(mlp["router"]["top"]), ff=int(mlp["expert"]["ff"]))
+        layers.append(StackLayerSpec(mixer, mlp))
+    return StackConfig(name=name, architecture="Lederax", vocab_size=int(doc["vocab"]), d_model=int(doc["width"]),
+                       layers=tuple(layers), embed_scale=float(doc["embedding"]["scale"]), norm_eps=float(doc["norm"]["eps"]),
+                       norm_groups=int(doc["norm"].get("groups", 1))).validate()
+
+
+def lederax_config_to_dict(cfg: StackConfig) -> Dict:
+    layers = []
+    for layer in cfg.layers:
+        m, f = layer.mixer, layer.mlp
+        layers.append({"type": "attention",
+                       "mixer": {"heads": m.heads, "kv_heads": m.kv_heads, "dim": m.dim, "vdim": m.vdim, "scale": m.scale,
+                                 "mask": None if m.window is None else {"size": m.window}, "v_mix": m.value_mix},
+                       "mlp": None if f is None else {"kind": "moe", "expert": {"ff": f.ff},
+                                                      "router": {"experts": f.experts, "top": f.top}}})
+    return {"architecture": "Lederax", "vocab": cfg.vocab_size, "width": cfg.d_model,
+            "embedding": {"scale": cfg.embed_scale}, "norm": {"eps": cfg.norm_eps, "groups": cfg.norm_groups}, "layers": layers}
+
+
+# architecture name in config.json -> (reader, writer)
+ARCHITECTURES = {"Lederax": (lederax_config_from_dict, lederax_config_to_dict)}
+
+
+def stack_config_from_dir(path) -> Optional[StackConfig]:
+    """The stack config of a checkpoint directory, or None when its config.json names no architecture of this kind."""
+    import json
+    from pathlib import Path
+
+    f = Path(path) / "config.json"
+    if not f.is_file():
+        return None
+    doc = json.loads(f.read_text())
+    arch = doc.get("architecture")
+    return ARCHITECTURES[arch][0](doc, name=Path(path).name) if arch in ARCHITECTURES else None
+
+
+def lederax_preset(name: str, d_model: int, n_layers: int, heads: int, kv_heads: int, dim: int, window: int, experts: int,
+                   top: int, ff: int, vocab_size: int, norm_groups: int = 2) -> StackConfig:
+    layer = StackLayerSpec(AttentionSpec(heads=heads, kv_heads=kv_heads, dim=dim, vdim=dim, scale=dim ** -0.5, window=window,
+                                         distance_bias=True, value_norm=True, value_mix=True, qkv_bias=True),
+                           MoESpec(experts=experts, top=top, ff=ff))
+    return StackConfig(name=name, architecture="Lederax", vocab_size=vocab_size, d_model=d_model, layers=(layer,) * n_layers,
+                       norm_groups=norm_groups).validate()
+
+
+def lederax_tiny_config(n_layers: int = 2, **kw) -> StackConfig:
+    """Toy model of the CPU tests and examples (byte-level tokenizer)."""
+    return replace(lederax_preset("lederax-tiny", d_model=96, n_layers=n_layers, heads=4, kv_heads=2, dim=24, window=20,
+                                  experts=6, top=2, ff=40, vocab_size=300), **kw)
+
+
+def lederax_8b_config(n_layers: int = 36, **kw) -> StackConfig:
+    """Layers as wide as Cosmos3-Nano's Reasoner tower, with as many active parameters a layer: attention 32 / 8 heads of
+    128, 4 of 32 experts of 4608 (up + down = the 3 x 12288 columns of a dense SwiGLU layer)."""
+    return replace(lederax_preset("lederax-8b", d_model=4096, n_layers=n_layers, heads=32, kv_heads=8, dim=128, window=4096,
+                                  experts=32, top=4, ff=4608, vocab_size=151936), **kw)
+
+
 MODEL_REGISTRY = {
+    "lederax-tiny": lederax_tiny_config,
+    "lederax-8b": lederax_8b_config,
     "tiny": tiny_config,
     "tiny128": tiny128_config,
     "Cosmos3-Nano": nano_config,
@@ -114,7 +271,8 @@ MODEL_REGISTRY = {
 }
 
 
-def get_model_config(name: str, **kw) -> MoTConfig:
+def get_model_config(name: str, **kw):
+    """MoTConfig (or StackConfig, for the decoder stacks) of a registered name."""
     key = name.rstrip("/").split("/")[-1] if name not in MODEL_REGISTRY else name
     if key not in MODEL_REGISTRY:
         raise KeyError(f"unknown model '{name}'; known: {sorted(MODEL_REGISTRY)}")

@@ -1,6 +1,7 @@
-"""Batched Reasoner decoding with tensor parallelism, a paged KV cache and CUDA graphs.
+"""Batched decoding: the Reasoner (`TPDecoder`) with tensor parallelism, a paged KV cache and CUDA graphs, and
+the config-declared decoder stacks (`StackDecoder`) on the same cache, step and sampler.
 
-One decode step for B sequences on each of `tp` ranks (heads and FFN units split by rank):
+One decode step of the Reasoner for B sequences on each of `tp` ranks (heads and FFN units split by rank):
   RMSNorm -> QKV split-K GEMM -> q/k RMSNorm + rotary -> KV-cache write -> paged-KV decode
   attention -> out-proj split-K GEMM -> one-shot all-reduce over NVLink -> (residual + RMSNorm
   fused) -> SwiGLU FC1 -> FC2 -> all-reduce -> ... -> final norm -> vocab-parallel LM head ->
@@ -21,7 +22,7 @@ import json
 import os
 import sys
 import time
-from typing import Dict, List, Optional
+from typing import Dict, List, Optional, Sequence, Tuple
 
 import torch
 import torch.distributed as dist
@@ -29,10 +30,113 @@ import torch.distributed as dist
 from .. import ops
 from ..config import MoTConfig, get_model_config
 from ..models import rope
+from ..models.stack import StackModel, StepBatch
+from ..ops.stack import make_tiles
 from .paged import PagedKVCache
 
 
-class TPDecoder:
+class StepDecoder:
+    """What every batched decoder shares: per-slot state in device tensors (tokens, lens, block table), the sampler, and the
+    step as one CUDA graph. A subclass sets `cfg`, `device`, `cache`, `page_size`, `tp`, `rank`, `group`, `v_loc` and
+    provides `_step_impl`, which consumes tokens / lens, writes next_tokens and advances lens."""
+
+    takes_portions = False   # prompts are prefilled in portions over the cache (StackDecoder), not by a separate forward
+
+    def _init_state(self) -> None:
+        self.graph = None
+        self.step_inc: Optional[torch.Tensor] = None  # int32 [B] of 0/1 set by the serving engine; None = all ones
+        self.sampling: Optional[Dict[str, torch.Tensor]] = None  # see enable_sampling
+        self.pos_delta: Optional[torch.Tensor] = None  # int64 [B]: rotary position minus cache position
+
+    def _step_impl(self) -> None:
+        raise NotImplementedError
+
+    def _finish_step(self, logits: torch.Tensor, b: int) -> None:
+        self.last_logits = logits                    # this rank's vocab shard, kept for inspection
+        if self.sampling is not None:
+            self._sample(logits)                     # global ids across the vocab shards, into self.next_tokens
+            return
+        val, idx = logits.float().max(dim=-1)
+        idx = idx + self.rank * self.v_loc
+        if self.tp > 1:
+            packed = torch.stack([val, idx.float()], dim=-1)      # [B, 2]
+            allp = torch.empty(self.tp * b, 2, device=self.device)            # rank-major concatenation
+            dist.all_gather_into_tensor(allp, packed, group=self.group)
+            allp = allp.view(self.tp, b, 2)
+            best = allp[..., 0].argmax(dim=0)
+            idx = allp[best, torch.arange(b, device=self.device), 1].long()
+        self.next_tokens.copy_(idx.clamp(max=self.cfg.vocab_size - 1))
+
+    # ------------------------------------------------------------------ sampling
+    SAMPLE_K = ops.SAMPLE_K  # candidates kept per slot; a request's top_k is clamped to it
+
+    def enable_sampling(self, batch: int) -> None:
+        """Per-slot sampling state, all on the device so that the step stays one CUDA graph:
+        temperature (0 = greedy), top_k, top_p, presence / repetition penalty, `seen_out` / `seen_any`
+        ([B, V] flags of tokens generated / seen in prompt or output) and a buffer of uniform noise that
+        the host refills before every step (the Gumbel-max draw inside the graph then needs no generator)."""
+        dev, v = self.device, self.v_loc  # `seen_*` cover this rank's vocabulary shard
+        self.sampling = {
+            "temperature": torch.zeros(batch, device=dev), "top_k": torch.ones(batch, dtype=torch.long, device=dev),
+            "top_p": torch.ones(batch, device=dev), "presence": torch.zeros(batch, device=dev),
+            "repetition": torch.ones(batch, device=dev),
+            "seen_out": torch.zeros(batch, v, dtype=torch.bool, device=dev),
+            "seen_any": torch.zeros(batch, v, dtype=torch.bool, device=dev),
+            "noise": torch.full((batch, self.SAMPLE_K), 0.5, device=dev),
+        }
+
+    def refill_noise(self, generator: Optional[torch.Generator] = None) -> None:
+        if self.sampling is not None:
+            self.sampling["noise"].uniform_(1e-7, 1.0, generator=generator)
+
+    def _sample(self, logits: torch.Tensor) -> torch.Tensor:
+        """Penalties, top-k / top-p and the Gumbel-max draw for every slot (`ops.sample_topk`, `ops.sample_pick`):
+        the 64 best penalised logits of this rank's vocabulary shard, the candidates of all shards gathered, then
+        the draw. Every rank ends up with the same choice (same candidates, same noise). The token consumed by
+        this step (self.tokens) counts as generated. Writes self.next_tokens."""
+        sp = self.sampling
+        cand = ops.sample_topk(logits, sp["seen_any"], sp["seen_out"], self.tokens, sp["presence"], sp["repetition"],
+                               self.rank * self.v_loc)
+        if self.tp > 1:
+            allc = torch.empty(self.tp * cand.shape[0], ops.SAMPLE_K, 2, device=cand.device)  # rank-major
+            dist.all_gather_into_tensor(allc, cand, group=self.group)
+            cand = allc
+        return ops.sample_pick(cand, self.tp, sp["temperature"], sp["top_k"], sp["top_p"], sp["noise"],
+                               self.cfg.vocab_size, self.next_tokens)
+
+    # ------------------------------------------------------------------ stepping
+    @torch.no_grad()
+    def step(self) -> torch.Tensor:
+        """One decode step for the whole batch; returns the new tokens [B] (device tensor)."""
+        if self.graph is not None:
+            self.graph.replay()
+        else:
+            self._step_impl()
+        self.tokens.copy_(self.next_tokens)
+        return self.next_tokens
+
+    @torch.no_grad()
+    def capture(self, warmup: int = 2) -> None:
+        """Captures `_step_impl` into a CUDA graph. Warm-up steps run first (workspace and
+        symmetric-memory set-up must not happen during capture); they advance the sequences."""
+        side = torch.cuda.Stream()
+        side.wait_stream(torch.cuda.current_stream())
+        with torch.cuda.stream(side):
+            for _ in range(warmup):
+                self._step_impl()
+                self.tokens.copy_(self.next_tokens)
+        torch.cuda.current_stream().wait_stream(side)
+        torch.cuda.synchronize()
+        if self.tp > 1:
+            dist.barrier(group=self.group)
+        g = torch.cuda.CUDAGraph()
+        with torch.cuda.graph(g):
+            self._step_impl()
+        self.graph = g
+        self.tokens.copy_(self.next_tokens)  # the capture ran one real step as well
+
+
+class TPDecoder(StepDecoder):
     def __init__(self, cfg: MoTConfig, tp: int, rank: int, group, device, page_size: int = 32,
                  max_batch: int = 32, max_len: int = 9000, seed: int = 0, fused: bool = True, dtype=torch.bfloat16):
         assert cfg.n_heads % tp == 0 and cfg.n_kv_heads % tp == 0 and cfg.ffn_dim % tp == 0
@@ -81,10 +185,7 @@ class TPDecoder:
             from ..parallel.tp import TPContext
             ranks = list(range(tp)) if group is None else dist.get_process_group_ranks(group)
             self._tpctx = TPContext(cfg, group, ranks, self.device, fused=self.fused, sequence_parallel=False)
-        self.graph = None
-        self.step_inc: Optional[torch.Tensor] = None  # int32 [B] of 0/1 set by the serving engine; None = all ones
-        self.sampling: Optional[Dict[str, torch.Tensor]] = None  # see enable_sampling
-        self.pos_delta: Optional[torch.Tensor] = None  # int64 [B]: rotary position minus cache position
+        self._init_state()
 
     # ------------------------------------------------------------------ helpers
     def _allreduce(self, x: torch.Tensor) -> torch.Tensor:
@@ -194,59 +295,6 @@ class TPDecoder:
             h, _ = ops.rmsnorm(delta, self.final_norm, self.cfg.rms_eps, residual=x)
         return ops.gemm(h, self.lm_head)             # [B, V/tp]
 
-    def _finish_step(self, logits: torch.Tensor, b: int) -> None:
-        self.last_logits = logits                    # this rank's vocab shard, kept for inspection
-        if self.sampling is not None:
-            self._sample(logits)                     # global ids across the vocab shards, into self.next_tokens
-            return
-        val, idx = logits.float().max(dim=-1)
-        idx = idx + self.rank * self.v_loc
-        if self.tp > 1:
-            packed = torch.stack([val, idx.float()], dim=-1)      # [B, 2]
-            allp = torch.empty(self.tp * b, 2, device=self.device)            # rank-major concatenation
-            dist.all_gather_into_tensor(allp, packed, group=self.group)
-            allp = allp.view(self.tp, b, 2)
-            best = allp[..., 0].argmax(dim=0)
-            idx = allp[best, torch.arange(b, device=self.device), 1].long()
-        self.next_tokens.copy_(idx.clamp(max=self.cfg.vocab_size - 1))
-
-    # ------------------------------------------------------------------ sampling (tp = 1)
-    SAMPLE_K = ops.SAMPLE_K  # candidates kept per slot; a request's top_k is clamped to it
-
-    def enable_sampling(self, batch: int) -> None:
-        """Per-slot sampling state, all on the device so that the step stays one CUDA graph:
-        temperature (0 = greedy), top_k, top_p, presence / repetition penalty, `seen_out` / `seen_any`
-        ([B, V] flags of tokens generated / seen in prompt or output) and a buffer of uniform noise that
-        the host refills before every step (the Gumbel-max draw inside the graph then needs no generator)."""
-        dev, v = self.device, self.v_loc  # `seen_*` cover this rank's vocabulary shard
-        self.sampling = {
-            "temperature": torch.zeros(batch, device=dev), "top_k": torch.ones(batch, dtype=torch.long, device=dev),
-            "top_p": torch.ones(batch, device=dev), "presence": torch.zeros(batch, device=dev),
-            "repetition": torch.ones(batch, device=dev),
-            "seen_out": torch.zeros(batch, v, dtype=torch.bool, device=dev),
-            "seen_any": torch.zeros(batch, v, dtype=torch.bool, device=dev),
-            "noise": torch.full((batch, self.SAMPLE_K), 0.5, device=dev),
-        }
-
-    def refill_noise(self, generator: Optional[torch.Generator] = None) -> None:
-        if self.sampling is not None:
-            self.sampling["noise"].uniform_(1e-7, 1.0, generator=generator)
-
-    def _sample(self, logits: torch.Tensor) -> torch.Tensor:
-        """Penalties, top-k / top-p and the Gumbel-max draw for every slot (`ops.sample_topk`, `ops.sample_pick`):
-        the 64 best penalised logits of this rank's vocabulary shard, the candidates of all shards gathered, then
-        the draw. Every rank ends up with the same choice (same candidates, same noise). The token consumed by
-        this step (self.tokens) counts as generated. Writes self.next_tokens."""
-        sp = self.sampling
-        cand = ops.sample_topk(logits, sp["seen_any"], sp["seen_out"], self.tokens, sp["presence"], sp["repetition"],
-                               self.rank * self.v_loc)
-        if self.tp > 1:
-            allc = torch.empty(self.tp * cand.shape[0], ops.SAMPLE_K, 2, device=cand.device)  # rank-major
-            dist.all_gather_into_tensor(allc, cand, group=self.group)
-            cand = allc
-        return ops.sample_pick(cand, self.tp, sp["temperature"], sp["top_k"], sp["top_p"], sp["noise"],
-                               self.cfg.vocab_size, self.next_tokens)
-
     # ------------------------------------------------------------------ public
     @torch.no_grad()
     def prefill_synthetic(self, batch: int, prompt_len: int, new_tokens: int, seed: int = 1) -> None:
@@ -326,35 +374,92 @@ class TPDecoder:
         self.embed = model.embed.data
         self.final_norm = model.ar_norm.data
 
-    @torch.no_grad()
-    def step(self) -> torch.Tensor:
-        """One decode step for the whole batch; returns the new tokens [B] (device tensor)."""
-        if self.graph is not None:
-            self.graph.replay()
+
+class StackDecoder(StepDecoder):
+    """Decoder of a config-declared layer stack (models/stack.py) over the paged cache, on one GPU. Decode steps run through
+    the shared step / graph machinery; prompts run in portions (`run_portions`): any number of sequences with any number of
+    new tokens each, against what earlier portions left in the cache."""
+
+    takes_portions = True
+
+    def __init__(self, model, page_size: int = 32, max_batch: int = 32, max_len: int = 9000, num_pages: Optional[int] = None):
+        self.model, self.cfg, self.device = model, model.cfg, model.device
+        self.tp, self.rank, self.group, self.v_loc = 1, 0, None, model.cfg.vocab_size
+        self.page_size = page_size
+        pages_per_seq = (max_len + page_size - 1) // page_size
+        self.cache = PagedKVCache(self.cfg.n_layers, 0, 0, num_pages or max_batch * pages_per_seq + 1, page_size,
+                                  pages_per_seq, model.dtype, self.device, kv_shapes=model.kv_shapes())
+        self.tile_sizes = model.tile_sizes(page_size)
+        self._init_state()
+
+    def _step_impl(self) -> None:
+        pos = self.lens.long()
+        slots = PagedKVCache.slots(self.table, pos[:, None], self.page_size)[:, 0].contiguous()
+        # attention sees the token being written; idle slots (length 0, no advance) see nothing
+        if self.step_inc is None:
+            self.lens.add_(1)
         else:
-            self._step_impl()
-        self.tokens.copy_(self.next_tokens)
-        return self.next_tokens
+            self.lens.add_(self.step_inc)
+        batch = StepBatch(self.tokens, slots, self.table, lens=self.lens, max_len=self.max_len)
+        self._finish_step(self.model.forward_step(batch, self.cache, self.tile_sizes), self.tokens.shape[0])
 
     @torch.no_grad()
-    def capture(self, warmup: int = 2) -> None:
-        """Captures `_step_impl` into a CUDA graph. Warm-up steps run first (workspace and
-        symmetric-memory set-up must not happen during capture); they advance the sequences."""
-        side = torch.cuda.Stream()
-        side.wait_stream(torch.cuda.current_stream())
-        with torch.cuda.stream(side):
-            for _ in range(warmup):
-                self._step_impl()
-                self.tokens.copy_(self.next_tokens)
-        torch.cuda.current_stream().wait_stream(side)
-        torch.cuda.synchronize()
-        if self.tp > 1:
-            dist.barrier(group=self.group)
-        g = torch.cuda.CUDAGraph()
-        with torch.cuda.graph(g):
-            self._step_impl()
-        self.graph = g
-        self.tokens.copy_(self.next_tokens)  # the capture ran one real step as well
+    def run_portions(self, entries: Sequence[Tuple[int, Sequence[int], int, Sequence[int]]],
+                     layers_out: Optional[list] = None) -> torch.Tensor:
+        """entries: (sequence id, its next tokens, how many it has in the cache already, places among these tokens whose
+        logits are wanted). The sequences' pages must have been reserved. Returns the wanted logits, in order."""
+        page, dev = self.page_size, self.device
+        seqs = [e[0] for e in entries]
+        counts = [len(e[1]) for e in entries]
+        table, _ = self.cache.host_tables(seqs)
+        toks = torch.tensor([t for e in entries for t in e[1]], dtype=torch.long)
+        if toks.numel() and not 0 <= int(toks.min()) <= int(toks.max()) < self.cfg.vocab_size:
+            raise ValueError("token id outside the vocabulary")
+        pos = torch.cat([torch.arange(e[2], e[2] + c) for e, c in zip(entries, counts)])
+        seq = torch.repeat_interleave(torch.arange(len(entries)), torch.tensor(counts))
+        slots = table[seq, pos // page].long() * page + pos % page
+        if bool((table[seq, pos // page] < 0).any()):
+            raise ValueError("a portion reaches beyond the pages reserved for its sequence")
+        row0 = [sum(counts[:i]) for i in range(len(counts))]
+        rows = [row0[i] + w for i, e in enumerate(entries) for w in e[3]]
+        batch = StepBatch(toks.to(dev), slots.to(dev), table.to(dev))
+        if all(c == 1 for c in counts):   # one new token each: the decode kernels
+            lens = torch.tensor([e[2] + 1 for e in entries], dtype=torch.int32)
+            batch.lens, batch.max_len = lens.to(dev), int(lens.max())
+        else:
+            portions = [(i, row0[i], counts[i], entries[i][2]) for i in range(len(entries))]
+            batch.tiles = {r: torch.tensor(make_tiles(portions, r), dtype=torch.int32).to(dev) for r in set(self.tile_sizes)}
+        sel = torch.tensor(rows, dtype=torch.long).to(dev)
+        return self.model.forward_step(batch, self.cache, self.tile_sizes, sel, layers_out)
+
+    @torch.no_grad()
+    def start_batch(self, prompts: Sequence[Sequence[int]], new_tokens: int, portion: int = 16384) -> None:
+        """Prefills one prompt per slot and readies a plain decode batch (the serving engine does its own admission)."""
+        last = []
+        self.seq_ids = list(range(len(prompts)))
+        for i, ids in enumerate(prompts):
+            self.cache.release(i)
+            assert self.cache.reserve(i, len(ids) + new_tokens), "KV pool exhausted"
+            for o in range(0, len(ids), portion):
+                part = ids[o:o + portion]
+                lg = self.run_portions([(i, part, o, [len(part) - 1] if o + len(part) == len(ids) else [])])
+            last.append(lg.float().argmax(-1))
+        self.table, _ = self.cache.tables(self.seq_ids)
+        self.lens = torch.tensor([len(p) for p in prompts], dtype=torch.int32, device=self.device)
+        self.max_len = max(len(p) for p in prompts) + new_tokens
+        self.tokens = torch.cat(last)
+        self.next_tokens = torch.zeros_like(self.tokens)
+
+
+def make_decoder(model, tp: int, rank: int, group, device, page_size: int, max_batch: int, max_len: int, dtype) -> StepDecoder:
+    """The decoder that serves `model`, holding its weights."""
+    if isinstance(model, StackModel):
+        if tp > 1:
+            raise ValueError("decoder stacks run on one GPU; start the engine without a tensor-parallel group")
+        return StackDecoder(model, page_size, max_batch, max_len)
+    dec = TPDecoder(model.cfg, tp, rank, group, device, page_size=page_size, max_batch=max_batch, max_len=max_len, dtype=dtype)
+    dec.load_from(model)
+    return dec
 
 
 def main(argv=None) -> int:

@@ -1,15 +1,18 @@
-"""Continuous batching for the Reasoner: requests join and leave a fixed set of decode slots while
+"""Continuous batching for the Reasoner and the decoder stacks: requests join and leave a fixed set of decode slots while
 the batch keeps stepping (the serving pattern behind the reference's published Reasoner numbers,
 which are measured through vLLM at client concurrency 1..256, reference
 inference_benchmarks.md:239-241,501-535).
 
-`BatchEngine` owns a `TPDecoder` whose batch is `max_batch` slots. A slot is either idle (length 0,
+`BatchEngine` owns a decoder (`make_decoder`) whose batch is `max_batch` slots. A slot is either idle (length 0,
 block table pointing at a scratch page, its lane of the step ignored) or bound to a request. Each
 engine step (1) admits waiting requests into idle slots while KV pages last — the prompts of the
 admitted group run through the AR tower in one padded forward and their K/V go into the requests' pages, (2) runs ONE decode step for all
 slots (the same CUDA graph whatever the mix of requests, because the per-slot state lives in device
 tensors that the host edits in place), (3) reads the new tokens back, appends them to their
 requests and retires the ones that hit an end token or their token limit, freeing pages and slot.
+Decoder stacks (`StackDecoder`) prefill in portions instead: an admitted request holds its slot and pages, and each engine
+step feeds up to `max_prefill_tokens` prompt tokens of the waiting prompts (several requests in one ragged forward, a long
+prompt over several steps) before the decode step of the requests that are already generating.
 Sampling (temperature, top-k, top-p, presence and repetition penalties, per request) runs on the device
 inside the same graph; temperature 0 is greedy.
 
@@ -28,9 +31,8 @@ from typing import Deque, Dict, List, Optional, Sequence
 import torch
 
 from .. import ops
-from ..config import MoTConfig
 from ..models import rope
-from .decoder import TPDecoder
+from .decoder import make_decoder
 from .paged import PagedKVCache
 
 
@@ -54,6 +56,7 @@ class Request:
     on_token: Optional[object] = None   # callable(token id), called from the engine thread for every new token
     out: List[int] = field(default_factory=list)
     slot: int = -1
+    prefilled: int = 0             # prompt tokens in the cache (decoders that take portions)
     t_submit: float = 0.0
     t_first: float = 0.0
     t_done: float = 0.0
@@ -63,13 +66,13 @@ class Request:
 
 class BatchEngine:
     def __init__(self, model, max_batch: int = 8, max_len: int = 4096, page_size: int = 32, device=None,
-                 dtype=None, use_graph: Optional[bool] = None, group=None):
-        """`group`: tensor-parallel process group (None = one rank). Every rank of the group builds the engine on
+                 dtype=None, use_graph: Optional[bool] = None, group=None, max_prefill_tokens: int = 16384):
+        """`max_prefill_tokens`: prompt tokens per forward. `group`: tensor-parallel process group (None = one rank). Every rank of the group builds the engine on
         the same model weights; rank 0 of the group takes the requests (`submit`), the others call `follow()`."""
         import torch.distributed as dist
 
         self.model = model
-        self.cfg: MoTConfig = model.cfg
+        self.cfg = model.cfg
         p = next(model.parameters())
         self.device = torch.device(device) if device is not None else p.device
         dtype = dtype or p.dtype
@@ -79,9 +82,7 @@ class BatchEngine:
         self.rank = dist.get_rank(group) if group is not None else 0
         self._new: List[dict] = []      # requests submitted on rank 0 since the last step (sent to the followers)
         self._stop = False
-        self.dec = TPDecoder(self.cfg, self.tp, self.rank, group, self.device, page_size=page_size, max_batch=max_batch,
-                             max_len=max_len, dtype=dtype)
-        self.dec.load_from(model)
+        self.dec = make_decoder(model, self.tp, self.rank, group, self.device, page_size, max_batch, max_len, dtype)
         cache = self.dec.cache
         # one page is set aside for idle slots: their (ignored) K/V writes land there
         self.scratch_seq = -1
@@ -104,7 +105,9 @@ class BatchEngine:
         self.finished: Dict[int, Request] = {}
         self._next_rid = 0
         self.steps = 0
-        self.max_prefill_tokens = 16384  # padded prompt tokens per prefill forward
+        # prompt tokens per prefill forward (padded ones for the Reasoner, the portions' own for a decoder stack)
+        self.max_prefill_tokens = max_prefill_tokens
+        self.prefilling: Deque[Request] = deque()   # requests that hold a slot but whose prompt is not in the cache yet
         self.use_graph = (self.device.type == "cuda") if use_graph is None else use_graph
         self._graph_ready = False
 
@@ -116,6 +119,8 @@ class BatchEngine:
                deepstack: Optional[Sequence[torch.Tensor]] = None, on_token=None) -> Request:
         if len(ids) < 1:
             raise ValueError("empty prompt")
+        if embeds is not None and self.dec.takes_portions:
+            raise ValueError("this model takes token prompts only (no media)")
         if len(ids) + max_new_tokens > self.max_len:
             raise ValueError(f"prompt ({len(ids)}) + max_new_tokens ({max_new_tokens}) exceeds max_len {self.max_len}")
         params = dict(ids=[min(int(t), self.cfg.vocab_size - 1) for t in ids], max_new_tokens=int(max_new_tokens),
@@ -206,8 +211,6 @@ class BatchEngine:
             h, kvs = self.model.ar_forward(self.model.embed_tokens(ids), rope.text_positions(n_max, 0, dev))
             delta = [0] * bsz
         table, _ = cache.tables([r.rid for r in group])
-        slot_idx = torch.tensor(slots, dtype=torch.long, device=dev)
-        dec.table[slot_idx] = table
         len_t = torch.tensor(lens, device=dev)
         pos = torch.arange(n_max, device=dev)[None].expand(bsz, -1)
         real = pos < len_t[:, None]                                          # [B, n_max]
@@ -218,6 +221,21 @@ class BatchEngine:
             cache.write(li, k[real][:, hs].contiguous(), v[real][:, hs].contiguous(), rows)
         last = h[torch.arange(bsz, device=dev), len_t - 1][:, None]          # [B, 1, d]
         logits = self.model.lm_logits(last).float()[:, 0]                    # [B, V]
+        self._start_decoding(group, slots, table, logits, delta)
+
+    def _start_decoding(self, group: List[Request], slots: List[int], table: torch.Tensor, logits: torch.Tensor,
+                        delta: List[int]) -> None:
+        """Binds prefilled requests to their decode slots and draws their first tokens from `logits` [B, V] fp32."""
+        dec, dev = self.dec, self.device
+        bsz, lens = len(group), [len(r.ids) for r in group]
+        slot_idx = torch.tensor(slots, dtype=torch.long, device=dev)
+        len_t = torch.tensor(lens, device=dev)
+        ids = torch.zeros(bsz, max(lens), dtype=torch.long)
+        for i, r in enumerate(group):
+            ids[i, :lens[i]] = torch.tensor(r.ids, dtype=torch.long)
+        ids = ids.to(dev)
+        real = torch.arange(max(lens), device=dev)[None] < len_t[:, None]
+        dec.table[slot_idx] = table
         # per-slot sampling state; the prompt tokens count as "seen" for the repetition penalty
         sp = dec.sampling
         for name, vals in (("temperature", [r.temperature for r in group]), ("top_p", [r.top_p for r in group]),
@@ -225,8 +243,8 @@ class BatchEngine:
                            ("repetition", [r.repetition_penalty for r in group])):
             sp[name][slot_idx] = torch.tensor(vals, dtype=torch.float32, device=dev)
         sp["top_k"][slot_idx] = torch.tensor([r.top_k for r in group], dtype=torch.long, device=dev)
-        seen = torch.zeros(bsz, dec.v_loc * self.tp, dtype=torch.bool, device=dev)   # whole (padded) vocabulary
-        seen.scatter_(1, ids, real)
+        # whole (padded) vocabulary; added up, because a padding position (id 0) must not clear the flag of a real token 0
+        seen = torch.zeros(bsz, dec.v_loc * self.tp, dtype=torch.int32, device=dev).scatter_add_(1, ids, real.int()) > 0
         sp["seen_any"][slot_idx] = seen[:, self.rank * dec.v_loc:(self.rank + 1) * dec.v_loc]
         sp["seen_out"][slot_idx] = False
         first = self._first_tokens(logits, slot_idx, seen[:, :logits.shape[1]])
@@ -236,7 +254,7 @@ class BatchEngine:
         dec.step_inc[slot_idx] = 1
         now = time.time()
         for r, slot, tok in zip(group, slots, first.tolist()):
-            r.slot, r.t_first = slot, now
+            r.slot, r.t_first, r.prefilled = slot, now, len(r.ids)
             self.slots[slot] = r
             self._accept(r, int(tok))
 
@@ -281,13 +299,8 @@ class BatchEngine:
         if r.future is not None and not r.future.done():
             r.future.set_result(r)
 
-    # ------------------------------------------------------------------ one engine step
-    @torch.no_grad()
-    def step(self) -> List[Request]:
-        """Admits what fits, runs one decode step for the batch, returns the requests that finished."""
-        done_before = set(self.finished)
-        if self.tp > 1:
-            self._sync_requests()
+    def _admit_waiting(self) -> None:
+        """Admits groups of waiting requests into free slots, each group prefilled in one padded forward."""
         cache = self.dec.cache
         free = [i for i in range(self.max_batch) if self.slots[i] is None]
         while self.waiting and free:
@@ -313,14 +326,63 @@ class BatchEngine:
             free = [i for i in range(self.max_batch) if self.slots[i] is None]
             if self.waiting and not cache.alloc.can_allocate(len(self.waiting[0].ids) + self.waiting[0].max_new_tokens):
                 break
-        if any(s is not None for s in self.slots):
+
+    @torch.no_grad()
+    def _prefill_portions(self) -> None:
+        """Hands slots and pages to waiting requests, then feeds up to `max_prefill_tokens` of the prompts that are not in
+        the cache yet, oldest first; requests whose prompt is complete draw their first token and start decoding."""
+        dec, cache = self.dec, self.dec.cache
+        for slot in range(self.max_batch):
+            if self.slots[slot] is not None or not self.waiting:
+                continue
+            r = self.waiting[0]
+            if not cache.reserve(r.rid, len(r.ids) + r.max_new_tokens):
+                break  # pages are short: the request stays first in line until others retire
+            self.waiting.popleft()
+            r.slot = slot
+            self.slots[slot] = r
+            self.prefilling.append(r)
+        budget, entries, done = self.max_prefill_tokens, [], []
+        for r in self.prefilling:
+            take = min(budget, len(r.ids) - r.prefilled)
+            if take <= 0:
+                break
+            full = r.prefilled + take == len(r.ids)
+            entries.append((r.rid, r.ids[r.prefilled:r.prefilled + take], r.prefilled, [take - 1] if full else []))
+            r.prefilled += take
+            budget -= take
+            if full:
+                done.append(r)
+        if not entries:
+            return
+        logits = dec.run_portions(entries)
+        for _ in done:
+            self.prefilling.popleft()
+        if done:
+            table, _ = cache.tables([r.rid for r in done])
+            # pages that a slot does not own read as the scratch page
+            table = torch.where(table < 0, torch.full_like(table, self.scratch_page), table)
+            self._start_decoding(done, [r.slot for r in done], table, logits.float(), [0] * len(done))
+
+    # ------------------------------------------------------------------ one engine step
+    @torch.no_grad()
+    def step(self) -> List[Request]:
+        """Admits what fits, runs one decode step for the batch, returns the requests that finished."""
+        done_before = set(self.finished)
+        if self.tp > 1:
+            self._sync_requests()
+        if self.dec.takes_portions:
+            self._prefill_portions()
+        else:
+            self._admit_waiting()
+        if any(s is not None and s.prefilled >= len(s.ids) for s in self.slots):
             if self.use_graph and not self._graph_ready:
                 self._capture()
             self.dec.refill_noise(self.noise_gen)
             new = self.dec.step().tolist()  # one device-to-host read per step (end-token detection)
             self.steps += 1
             for slot, r in enumerate(self.slots):
-                if r is not None:
+                if r is not None and r.prefilled >= len(r.ids):
                     self._accept(r, int(new[slot]))
         return [self.finished[k] for k in self.finished if k not in done_before]
 
@@ -391,6 +453,7 @@ class EngineWorker:
                     if r.future is not None and not r.future.done():
                         r.future.set_exception(e)
                 eng.waiting.clear()
+                eng.prefilling.clear()
                 for s, r in enumerate(eng.slots):
                     if r is not None:
                         eng.slots[s] = None
@@ -406,9 +469,10 @@ def main(argv=None) -> int:
 
     from ..config import get_model_config
     from ..models.mot import MoTModel
+    from ..models.stack import is_stack_name, load_stack
 
     ap = argparse.ArgumentParser(description=main.__doc__)
-    ap.add_argument("--model", default="Cosmos3-Nano")
+    ap.add_argument("--model", default="Cosmos3-Nano", help="registered name, or a decoder stack's checkpoint directory")
     ap.add_argument("--requests", type=int, default=256)
     ap.add_argument("--max-num-seqs", type=int, default=64)
     ap.add_argument("--prompt-len", type=int, default=306, help="50 text tokens + a short clip's vision tokens")
@@ -420,9 +484,14 @@ def main(argv=None) -> int:
     cuda = torch.cuda.is_available()
     dev = torch.device("cuda", 0) if cuda else torch.device("cpu")
     dtype = torch.bfloat16 if cuda else torch.float32
-    cfg = get_model_config(args.model, **({"n_layers": args.layers} if args.layers else {}))
-    model = MoTModel(cfg, dtype=dtype, device=dev, towers=("ar",))  # the Reasoner needs the AR tower only
-    model.init_weights(seed=0)
+    layers = {"n_layers": args.layers} if args.layers else {}
+    if is_stack_name(args.model):
+        model = load_stack(args.model, dtype, dev, **layers)
+        cfg = model.cfg
+    else:
+        cfg = get_model_config(args.model, **layers)
+        model = MoTModel(cfg, dtype=dtype, device=dev, towers=("ar",))  # the Reasoner needs the AR tower only
+        model.init_weights(seed=0)
     eng = BatchEngine(model, max_batch=args.max_num_seqs, max_len=args.prompt_len + args.new_tokens + 16,
                       page_size=args.page_size)
     g = torch.Generator().manual_seed(0)

@@ -1,15 +1,16 @@
-"""Paged KV cache of the Reasoner: fixed-size pages per layer, a native (C++) block allocator
+"""Paged KV cache of the Reasoner and the decoder stacks: fixed-size pages per layer, a native (C++) block allocator
 that owns the page tables, and device-side tables that the decode-attention kernel reads.
 
 Layout per layer: k_cache, v_cache [num_pages, Hkv_local, page_size, head_dim] bf16 (the rows of one
 (page, head) are contiguous, which is what the decode kernel streams). A sequence
 owns a list of pages; token i of the sequence lives in page table[i // page_size] at offset
-i % page_size. Pages for the whole generation (prompt + max new tokens) can be reserved up front,
+i % page_size. Layers may differ in heads and head sizes, keys and values too (`kv_shapes`); the page tables are shared
+by all layers. Pages for the whole generation (prompt + max new tokens) can be reserved up front,
 which keeps the block table static during decode (a requirement for CUDA-graph replay).
 """
 from __future__ import annotations
 
-from typing import Sequence
+from typing import Optional, Sequence, Tuple
 
 import torch
 
@@ -69,12 +70,14 @@ def make_allocator(num_blocks: int, block_size: int, max_blocks_per_seq: int):
 
 class PagedKVCache:
     def __init__(self, n_layers: int, n_kv_heads: int, head_dim: int, num_pages: int, page_size: int,
-                 max_pages_per_seq: int, dtype=torch.bfloat16, device="cuda"):
+                 max_pages_per_seq: int, dtype=torch.bfloat16, device="cuda",
+                 kv_shapes: Optional[Sequence[Tuple[int, int, int]]] = None):
+        """`kv_shapes`: (kv heads, key size, value size) of every layer; None = n_kv_heads x head_dim throughout."""
         self.n_layers, self.page_size, self.max_pages = n_layers, page_size, max_pages_per_seq
         self.alloc = make_allocator(num_pages, page_size, max_pages_per_seq)
-        shape = (num_pages, n_kv_heads, page_size, head_dim)
-        self.k = [torch.zeros(shape, dtype=dtype, device=device) for _ in range(n_layers)]
-        self.v = [torch.zeros(shape, dtype=dtype, device=device) for _ in range(n_layers)]
+        shapes = list(kv_shapes) if kv_shapes is not None else [(n_kv_heads, head_dim, head_dim)] * n_layers
+        self.k = [torch.zeros((num_pages, h, page_size, kd), dtype=dtype, device=device) for h, kd, _ in shapes]
+        self.v = [torch.zeros((num_pages, h, page_size, vd), dtype=dtype, device=device) for h, _, vd in shapes]
         self.device = torch.device(device)
 
     def reserve(self, seq_id: int, tokens: int) -> bool:
@@ -86,10 +89,15 @@ class PagedKVCache:
 
     def tables(self, seq_ids: Sequence[int]):
         """(block_table [n, max_pages] int32, reserved lengths [n] int32) on the cache's device."""
+        t, l = self.host_tables(seq_ids)
+        return t.to(self.device), l.to(self.device)
+
+    def host_tables(self, seq_ids: Sequence[int]):
+        """The same on the host (unused entries -1)."""
         t = torch.empty(len(seq_ids), self.max_pages, dtype=torch.int32)
         l = torch.empty(len(seq_ids), dtype=torch.int32)
         self.alloc.fill_tables(list(seq_ids), t, l)
-        return t.to(self.device), l.to(self.device)
+        return t, l
 
     @staticmethod
     def slots(table: torch.Tensor, positions: torch.Tensor, page_size: int) -> torch.Tensor:

@@ -458,7 +458,9 @@ flash_attn_fwd_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
 #pragma unroll
         for (int i = 8; i < 128; i += 16)
 #pragma unroll
-          for (int e = 0; e < 8; ++e) mx8[e] = max3(mx8[e], __uint_as_float(s[i + e]), __uint_as_float(s[i + 8 + e]));
+          for (int e = 0; e < 8; ++e)
+            mx8[e] = i + 8 < 128 ? max3(mx8[e], __uint_as_float(s[i + e]), __uint_as_float(s[(i + 8 + e) & 127]))
+                                 : fmaxf(mx8[e], __uint_as_float(s[i + e]));   // the last eight have no partner
       }
       const float mx = max3(max3(mx8[0], mx8[1], mx8[2]), max3(mx8[3], mx8[4], mx8[5]), fmaxf(mx8[6], mx8[7]));
       const float m_new = fmaxf(m_used, mx * sl2);

@@ -13,6 +13,21 @@
 #include "kernels.h"
 #include "runtime.h"
 
+namespace cosmos {
+// One int32 status word per device; kernels CAS their first failure code into it.
+at::Tensor status_tensor(int device) {
+  static std::mutex mu;
+  static std::map<int, at::Tensor> words;
+  std::lock_guard<std::mutex> g(mu);
+  auto it = words.find(device);
+  if (it == words.end()) {
+    at::Tensor t = at::zeros({1}, at::TensorOptions().dtype(at::kInt).device(at::kCUDA, device));
+    it = words.emplace(device, t).first;
+  }
+  return it->second;
+}
+}  // namespace cosmos
+
 namespace {
 constexpr int kDefaultAttnExpEmu = 0;
 
@@ -27,18 +42,7 @@ void check_bf16_cuda(const Tensor& t, const char* name) {
 }
 const void* opt_ptr(const OptT& t) { return t.has_value() && t->defined() ? t->data_ptr() : nullptr; }
 
-// One int32 status word per device; kernels CAS their first failure code into it.
-Tensor status_tensor(int device) {
-  static std::mutex mu;
-  static std::map<int, Tensor> words;
-  std::lock_guard<std::mutex> g(mu);
-  auto it = words.find(device);
-  if (it == words.end()) {
-    Tensor t = at::zeros({1}, at::TensorOptions().dtype(at::kInt).device(at::kCUDA, device));
-    it = words.emplace(device, t).first;
-  }
-  return it->second;
-}
+using cosmos::status_tensor;
 
 Tensor status_word() {
   int dev = 0;

@@ -46,6 +46,11 @@ enum : int {
   SITE_DECODE_POST_SLOT = 2,
   SITE_PAGED_DECODE_PAGE = 3,
   SITE_PAGED_DECODE_TC_PAGE = 4,
+  SITE_STACK_TOKEN = 5,   // token id of a layer stack's step
+  SITE_STACK_SLOT = 6,    // cache slot of a layer stack's step
+  SITE_STACK_PAGE = 7,    // page id read by windowed attention
+  SITE_MOE_EXPERT = 8,    // expert id of a routing table
+  SITE_MOE_ROW = 9,       // row of the expert-sorted buffers
   SITE_SELFTEST = 15,
 };
 
@@ -395,6 +400,7 @@ __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
   __nv_bfloat162 t = __floats2bfloat162_rn(lo, hi);
   return *reinterpret_cast<uint32_t*>(&t);
 }
+__device__ __forceinline__ float gelu_erf(float z) { return 0.5f * z * (1.f + erff(z * 0.70710678118654752f)); }
 __device__ __forceinline__ float bf16lo(uint32_t u) { return __uint_as_float(u << 16); }
 __device__ __forceinline__ float bf16hi(uint32_t u) { return __uint_as_float(u & 0xFFFF0000u); }
 

@@ -9,12 +9,18 @@
 //
 // Fused epilogues (template parameter EPI):
 //   EPI_PLAIN        C = acc (+ bias)
+//   EPI_GELU         C = gelu(acc (+ bias)), the exact (erf) form
 //   EPI_SWIGLU       B holds [gate ; up] stacked along N; C[m, j] = silu(gate_j) * up_j  (N/2 wide)
 //   EPI_GATED_RESID  C = R + gate[m / rows_per_batch, n] * (acc + bias)   (AdaLN gated residual)
 //   EPI_QKV_ROPE     columns are heads of 128: per-head RMSNorm (q/k) + rotary embedding, and
 //                    each 128-column chunk is written through a routing table, so a chunk
 //                    can land in another GPU's buffer (sequence->head all-to-all of Ulysses
 //                    context parallelism done by the epilogue's stores).
+//
+// Grouped by a tile map (GemmParams::tile_map, mixture-of-experts layers): the rows of A are sorted by group, the map
+// names the group and the row range of every m-tile, and the group picks its N rows of B (the groups' weights stacked
+// along N). Segments are neither padded nor aligned: a tile's rows beyond its range are other groups' rows, computed
+// and not stored. The number of m-tiles lives on the device, so a captured graph follows the routing of each replay.
 //
 // All mbarrier waits are bounded; on expiry the kernel records a status code and exits
 // through the common tail (TMEM is freed).
@@ -77,6 +83,9 @@ struct GemmParams {
   int conv_cblocks;      // input channels / 64
   int conv_hp, conv_wp, conv_tpad;
   int conv_shift[27];    // row offset of each filter tap in the flattened padded volume
+  // grouped by a tile map (see the file comment): {group, first row, rows, unused} per m-tile; tile rows = TILE_M
+  const int4* tile_map;
+  const int* n_tiles_m;  // number of m-tiles of this launch (device)
   int debug;             // timing experiments (wrong results): 1 = every tile loads operand tile (0, 0); 2 = no loads at all
 };
 
@@ -98,6 +107,19 @@ __device__ __forceinline__ void tile_coords(int t, int m_tiles, int n_tiles, int
   const int r = t - band * GM * n_tiles;
   tm = first_m + r % band_m;
   tn = r / band_m;
+}
+
+// Row ranges of an m-tile: first row of A, end of the rows it owns, first row of its group's weights in B.
+struct TileRows {
+  int m0, m_end, b_row;
+};
+template <int TILE_M>
+__device__ __forceinline__ TileRows tile_rows(const GemmParams& p, int tm) {
+  if (p.tile_map) {
+    const int4 e = p.tile_map[tm];
+    return {e.y, e.y + e.z, e.x * p.N};
+  }
+  return {tm * TILE_M, p.M, 0};
 }
 
 template <int EPI, int NC>
@@ -131,7 +153,10 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
 
   const int warp = threadIdx.x >> 5;
   const int lane = threadIdx.x & 31;
-  const int total_tiles = g.total;
+  // the tile map's length is read before any programmatic-dependency wait: such launches are never programmatic
+  const int m_tiles0 = g.p[0].tile_map ? *g.p[0].n_tiles_m : g.p[0].m_tiles;
+  const int total_tiles = g.p[0].tile_map ? m_tiles0 * g.p[0].n_tiles * g.p[0].k_splits : g.total;
+  const int tiles0 = g.p[0].tile_map ? total_tiles : g.tiles0;
 
   int prefetched = 0;  // stages whose B half thread 0 has requested ahead of the producer loop
   if (threadIdx.x == 0) {
@@ -154,8 +179,8 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
     // Weight prefetch (single-CTA tiles, B in its [N, K] layout): the B halves of the first tile's first stages are
     // requested here, while warp 1 still allocates tensor memory and before the dependency wait of a programmatic
     // launch; their A halves follow in the producer loop. A stage's full barrier completes when both have landed.
-    if (NC == 1 && EPI != EPI_CONV && first_tile < total_tiles && first_tile < g.tiles0 && !g.p[0].b_mn &&
-        !g.p[0].debug) {
+    if (NC == 1 && EPI != EPI_CONV && first_tile < total_tiles && first_tile < tiles0 && !g.p[0].b_mn &&
+        !g.p[0].debug && !g.p[0].tile_map) {
       const GemmParams& p = g.p[0];
       const int k_blocks = (p.K + BK - 1) / BK;
       const int ks = first_tile % p.k_splits;
@@ -199,18 +224,19 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
       bool ok = true;
       pdl_wait();
       for (int t = first_tile; t < total_tiles && ok; t += tile_step) {
-        const int second = t >= g.tiles0;
+        const int second = t >= tiles0;
         const GemmParams& p = g.p[second];
         const CUtensorMap* mA = second ? &tmA1 : &tmA;
         const CUtensorMap* mB = second ? &tmB1 : &tmB;
         const int k_blocks = (p.K + BK - 1) / BK;
-        const int tl = second ? t - g.tiles0 : t;
+        const int tl = second ? t - tiles0 : t;
         const int ks = tl % p.k_splits;
         const int kb0 = ks * k_blocks / p.k_splits, kb1 = (ks + 1) * k_blocks / p.k_splits;
         int tm, tn;
-        tile_coords(tl / p.k_splits, p.m_tiles, p.n_tiles, tm, tn);
-        const int m0 = (p.debug & 1) ? 0 : tm * TILE_M + int(cta_rank) * BM;
-        const int n0 = (p.debug & 1) ? 0 : ((EPI == EPI_SWIGLU) ? tn * 128 : tn * BN);
+        tile_coords(tl / p.k_splits, second ? p.m_tiles : m_tiles0, p.n_tiles, tm, tn);
+        const TileRows tr = tile_rows<TILE_M>(p, tm);
+        const int m0 = (p.debug & 1) ? 0 : tr.m0 + int(cta_rank) * BM;
+        const int n0 = (p.debug & 1) ? 0 : tr.b_row + ((EPI == EPI_SWIGLU) ? tn * 128 : tn * BN);
         if (p.debug & 2) continue;
         for (int kb = kb0; kb < kb1; ++kb, ++it) {
           const int s = it % STAGES;
@@ -296,10 +322,10 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
       int it = 0, tcount = 0;
       bool ok = true;
       for (int t = first_tile; t < total_tiles && ok; t += tile_step, ++tcount) {
-        const int second = t >= g.tiles0;
+        const int second = t >= tiles0;
         const GemmParams& p = g.p[second];
         const int k_blocks = (p.K + BK - 1) / BK;
-        const int ks = (second ? t - g.tiles0 : t) % p.k_splits;
+        const int ks = (second ? t - tiles0 : t) % p.k_splits;
         const int kb0 = ks * k_blocks / p.k_splits, kb1 = (ks + 1) * k_blocks / p.k_splits;
         const int b = tcount & 1;
         const uint32_t bph = (tcount >> 1) & 1;
@@ -362,18 +388,19 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
     for (int t = first_tile; t < total_tiles; t += tile_step, ++tcount) {
       const int b = tcount & 1;
       const uint32_t bph = (tcount >> 1) & 1;
-      const int second = t >= g.tiles0;
+      const int second = t >= tiles0;
       const GemmParams& p = g.p[second];
-      const int tl = second ? t - g.tiles0 : t;
+      const int tl = second ? t - tiles0 : t;
       int tm, tn;
-      tile_coords(tl / p.k_splits, p.m_tiles, p.n_tiles, tm, tn);
-      const int m = tm * TILE_M + int(cta_rank) * BM + row_in_tile;
+      tile_coords(tl / p.k_splits, second ? p.m_tiles : m_tiles0, p.n_tiles, tm, tn);
+      const TileRows tr = tile_rows<TILE_M>(p, tm);
+      const int m = tr.m0 + int(cta_rank) * BM + row_in_tile;
       if (!mbar_wait(tfull_bar(b), bph, abort_flag, p.status, ST_TIMEOUT_EPI)) break;
       tc_fence_after();
       const uint32_t t_addr = tmem_base + (uint32_t(quad * 32) << 16) + b * BN;
-      const bool row_ok = m < p.M;
+      const bool row_ok = m < tr.m_end;
 
-      if ((EPI == EPI_PLAIN || EPI == EPI_SWIGLU || EPI == EPI_GATED_RESID) && p.k_splits > 1) {
+      if ((EPI == EPI_PLAIN || EPI == EPI_SWIGLU || EPI == EPI_GATED_RESID || EPI == EPI_GELU) && p.partial) {
         // raw fp32 partial sums; accumulator column c maps to output column col(c)
         float* dst_row = p.partial + ((long long)(tl % p.k_splits) * p.M + m) * p.N;
 #pragma unroll 1
@@ -398,7 +425,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
             }
           }
         }
-      } else if constexpr (EPI == EPI_PLAIN || EPI == EPI_GATED_RESID) {
+      } else if constexpr (EPI == EPI_PLAIN || EPI == EPI_GATED_RESID || EPI == EPI_GELU) {
         const int n0 = tn * BN;
 #pragma unroll 1
         for (int c = 0; c < BN; c += 32) {
@@ -415,6 +442,10 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
 #pragma unroll
               for (int i = 0; i < 32; ++i)
                 if (full32 || n + i < p.N) f[i] += __bfloat162float(p.bias[n + i]);
+            }
+            if constexpr (EPI == EPI_GELU) {
+#pragma unroll
+              for (int i = 0; i < 32; ++i) f[i] = gelu_erf(f[i]);
             }
             if constexpr (EPI == EPI_GATED_RESID) {
               const bf16* g = p.gate ? p.gate + (long long)(m / p.rows_per_batch) * p.N + n : nullptr;
@@ -810,6 +841,10 @@ splitk_reduce_kernel(const float* __restrict__ partial, int k_splits, int M, int
 #pragma unroll
         for (int e = 0; e < 4; ++e) f[e] += __bfloat162float(bias[n + e]);
       }
+      if (epi == EPI_GELU) {
+#pragma unroll
+        for (int e = 0; e < 4; ++e) f[e] = gelu_erf(f[e]);
+      }
       if (epi == EPI_GATED_RESID) {
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
@@ -978,7 +1013,7 @@ static void launch(const CUtensorMap* maps, const cb::GemmGroup& g, int units, i
   at[0].val.clusterDim.x = NC; at[0].val.clusterDim.y = 1; at[0].val.clusterDim.z = 1;
   at[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
   at[1].val.programmaticStreamSerializationAllowed = 1;
-  cfg.attrs = at; cfg.numAttrs = (NC == 1 && pdl_on()) ? 2 : 1;
+  cfg.attrs = at; cfg.numAttrs = (NC == 1 && pdl_on() && !g.p[0].tile_map) ? 2 : 1;
   cudaLaunchKernelEx(&cfg, cb::gemm_bf16_kernel<EPI, NC>, maps[0], maps[1], maps[2], maps[3], g);
 }
 
@@ -987,6 +1022,7 @@ static void launch_epi(int epi, const CUtensorMap* maps, const cb::GemmGroup& g,
                        cudaStream_t stream) {
   switch (epi) {
     case EPI_PLAIN: launch<EPI_PLAIN, NC>(maps, g, units, limit, stream); break;
+    case EPI_GELU: launch<EPI_GELU, NC>(maps, g, units, limit, stream); break;
     case EPI_SWIGLU: launch<EPI_SWIGLU, NC>(maps, g, units, limit, stream); break;
     case EPI_GATED_RESID: launch<EPI_GATED_RESID, NC>(maps, g, units, limit, stream); break;
     case EPI_QKV_ROPE: launch<EPI_QKV_ROPE, NC>(maps, g, units, limit, stream); break;
@@ -1005,7 +1041,7 @@ static void fill_problem(const GemmArgs& a, cb::GemmParams& p, CUtensorMap& ta, 
     throw std::runtime_error("gemm_bf16: SwiGLU epilogue needs N/2 to be a multiple of 8");
   if (a.epi == EPI_QKV_ROPE && a.N % 128 != 0)
     throw std::runtime_error("gemm_bf16: QKV epilogue needs N to be a multiple of 128");
-  if ((a.epi == EPI_PLAIN || a.epi == EPI_GATED_RESID || a.epi == EPI_CONV) && (a.ldc % 8 != 0))
+  if ((a.epi == EPI_PLAIN || a.epi == EPI_GELU || a.epi == EPI_GATED_RESID || a.epi == EPI_CONV) && (a.ldc % 8 != 0))
     throw std::runtime_error("gemm_bf16: ldc must be a multiple of 8");
   if (a.epi == EPI_CONV) {
     if (a.conv_c <= 0 || a.conv_c % 64 != 0 || a.K != 27 * a.conv_c || a.N % 32 != 0 || a.conv_hp < 3 ||
@@ -1016,7 +1052,7 @@ static void fill_problem(const GemmArgs& a, cb::GemmParams& p, CUtensorMap& ta, 
   const uint64_t dimsA[2] = {(uint64_t)(a.epi == EPI_CONV ? a.conv_c : a.K), (uint64_t)a.M};
   const uint64_t strA[1] = {(uint64_t)a.lda * 2};
   const uint32_t boxA[2] = {cb::BK, cb::BM};
-  const uint64_t dimsB[2] = {(uint64_t)a.K, (uint64_t)a.N};
+  const uint64_t dimsB[2] = {(uint64_t)a.K, (uint64_t)a.N * (uint64_t)(a.tile_map ? a.n_groups : 1)};
   const uint64_t strB[1] = {(uint64_t)a.ldb * 2};
   const uint32_t boxB[2] = {cb::BK, 128};
   if (a.a_mn) {
@@ -1073,6 +1109,14 @@ static void fill_problem(const GemmArgs& a, cb::GemmParams& p, CUtensorMap& ta, 
   p.k_splits = 1;
   p.partial = nullptr;
   p.debug = g_debug;
+  p.tile_map = reinterpret_cast<const int4*>(a.tile_map);
+  p.n_tiles_m = a.n_tiles_m;
+  if (a.tile_map) {
+    if (a.a_mn || a.b_mn || !a.n_tiles_m || a.n_groups < 1 || a.max_tiles_m < 1 || a.tile_m != cb::BM * nc ||
+        (a.epi != EPI_PLAIN && a.epi != EPI_GELU) || (long long)a.N * a.n_groups > 0x7fffffffll)
+      throw std::runtime_error("gemm_bf16: bad tile-map launch");
+    p.m_tiles = a.max_tiles_m;   // upper bound for the grid; the kernel reads the count
+  }
   if (a.epi == EPI_CONV) {
     p.conv_cblocks = a.conv_c / 64;
     p.conv_hp = a.conv_hp; p.conv_wp = a.conv_wp; p.conv_tpad = a.conv_tpad;
@@ -1089,7 +1133,7 @@ void gemm_set_cta_pair(bool on) { g_pair = on ? 1 : 0; }
 void gemm_set_debug(int bits) { g_debug = bits; }
 
 int gemm_pick_k_splits(int M, int N, int K, int epi) {
-  if (epi != EPI_PLAIN && epi != EPI_SWIGLU && epi != EPI_GATED_RESID) return 1;
+  if (epi != EPI_PLAIN && epi != EPI_SWIGLU && epi != EPI_GATED_RESID && epi != EPI_GELU) return 1;
   const int m_tiles = (M + cb::BM - 1) / cb::BM;
   const int n_tiles = epi == EPI_SWIGLU ? (N / 2 + 127) / 128 : (N + cb::BN - 1) / cb::BN;
   const int tiles = m_tiles * n_tiles;
@@ -1129,8 +1173,11 @@ void gemm_bf16_grouped(const GemmArgs* args, int n, cudaStream_t stream) {
   // CTA pairs (256-row tiles) as soon as a problem has more than one 128-row tile
   const bool two = n == 2 && args[1].M > 0;
   // (not for the SwiGLU epilogue: measured 3 - 10 % slower on pairs at 16384 x 24576 x 4096)
-  const int nc = (pair_enabled() && args[0].epi != EPI_SWIGLU && (args[0].M > cb::BM || (two && args[1].M > cb::BM)))
+  if (args[0].tile_map && two) throw std::runtime_error("gemm_bf16_grouped: a tile map takes one problem");
+  const int nc = args[0].tile_map ? args[0].tile_m / cb::BM
+                 : (pair_enabled() && args[0].epi != EPI_SWIGLU && (args[0].M > cb::BM || (two && args[1].M > cb::BM)))
                      ? 2 : 1;
+  if (nc != 1 && nc != 2) throw std::runtime_error("gemm_bf16_grouped: tile rows must be 128 or 256");
   cb::GemmGroup g{};
   CUtensorMap maps[4];
   fill_problem(args[0], g.p[0], maps[0], maps[1], nc);
@@ -1154,7 +1201,7 @@ void gemm_bf16_grouped(const GemmArgs* args, int n, cudaStream_t stream) {
 
 void gemm_bf16(const GemmArgs& a, cudaStream_t stream) {
   if (a.M <= 0 || a.N <= 0) return;
-  if (a.k_splits <= 1) {
+  if (a.k_splits <= 1 && !a.partial_only) {
     gemm_bf16_grouped(&a, 1, stream);
     return;
   }
@@ -1165,10 +1212,11 @@ void gemm_bf16(const GemmArgs& a, cudaStream_t stream) {
   CUtensorMap maps[4];
   // more than one 128-row tile (a serving batch of 256): CTA pairs, so that each CTA stages half of the weight tile
   // (the skinny GEMMs of such a batch are bound by operand delivery into shared memory, not by HBM)
-  const int nc = (pair_enabled() && a.epi != EPI_SWIGLU && a.M > cb::BM) ? 2 : 1;
+  const int nc = a.tile_map ? a.tile_m / cb::BM : (pair_enabled() && a.epi != EPI_SWIGLU && a.M > cb::BM) ? 2 : 1;
+  if (nc != 1 && nc != 2) throw std::runtime_error("gemm_bf16: tile rows must be 128 or 256");
   fill_problem(a, g.p[0], maps[0], maps[1], nc);
   const int k_blocks = (a.K + cb::BK - 1) / cb::BK;
-  const int ks = a.k_splits < k_blocks ? a.k_splits : k_blocks;
+  const int ks = a.k_splits < 1 ? 1 : a.k_splits < k_blocks ? a.k_splits : k_blocks;
   g.p[0].k_splits = ks;
   g.p[0].partial = a.partial;
   g.tiles0 = g.total = g.p[0].m_tiles * g.p[0].n_tiles * ks;
@@ -1177,12 +1225,14 @@ void gemm_bf16(const GemmArgs& a, cudaStream_t stream) {
   if (nc == 2) {
     switch (a.epi) {
       case EPI_PLAIN: launch<EPI_PLAIN, 2>(maps, g, g.total, 0, stream); break;
+      case EPI_GELU: launch<EPI_GELU, 2>(maps, g, g.total, 0, stream); break;
       case EPI_GATED_RESID: launch<EPI_GATED_RESID, 2>(maps, g, g.total, 0, stream); break;
       default: throw std::runtime_error("gemm_bf16: unknown epilogue");
     }
   } else {
     switch (a.epi) {
       case EPI_PLAIN: launch<EPI_PLAIN, 1>(maps, g, g.total, 0, stream); break;
+      case EPI_GELU: launch<EPI_GELU, 1>(maps, g, g.total, 0, stream); break;
       case EPI_SWIGLU: launch<EPI_SWIGLU, 1>(maps, g, g.total, 0, stream); break;
       case EPI_GATED_RESID: launch<EPI_GATED_RESID, 1>(maps, g, g.total, 0, stream); break;
       default: throw std::runtime_error("gemm_bf16: unknown epilogue");

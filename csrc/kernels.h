@@ -14,6 +14,7 @@ enum GemmEpilogue : int {
   EPI_ATTN_P = 5,
   // C = P[m, n] * (acc - D[m]) * scale, with P passed as the residual operand
   EPI_ATTN_DS = 6,
+  EPI_GELU = 7,  // C = gelu(acc (+ bias)), exact (erf) form
 };
 
 enum AttnMask : int {
@@ -76,6 +77,12 @@ struct GemmArgs {
   // the same padded positions; only interior rows (frame >= conv_tpad, 1 <= h <= hp-2,
   // 1 <= w <= wp-2) are written, so a zero border stays zero.
   int conv_c = 0, conv_hp = 0, conv_wp = 0, conv_tpad = 0;
+  // Grouped by a tile map (mixture of experts): A [M, K] holds its rows sorted by group, B [n_groups * N, K] the groups'
+  // weights stacked, tile_map[max_tiles_m] (device int4: group, first row, rows, -) the m-tiles of tile_m (128 or 256)
+  // rows, *n_tiles_m (device) how many of them there are. EPI_PLAIN / EPI_GELU only.
+  const void* tile_map = nullptr;
+  const int* n_tiles_m = nullptr;
+  int n_groups = 0, max_tiles_m = 0, tile_m = 128;
 };
 // Split count that fills the machine for a skinny problem (1 = do not split).
 int gemm_pick_k_splits(int M, int N, int K, int epi);

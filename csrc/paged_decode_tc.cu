@@ -18,9 +18,14 @@
 // already in flight while the current one finishes. Every wait is bounded.
 //
 //   k_cache / v_cache [num_pages, Hkv, page_size, 128] bf16, page_size in {8, 16, 32, 64, 128}
+//
+// WIN = true (window_attn_decode_tc, stack.h) adds a sliding window, a distance bias and head sizes up to 128 that are
+// multiples of 8 (k_cache [.., dim], v_cache [.., vdim]): only the pages that the window touches are read, a thread
+// subtracts its token's bias from the scores of the group's heads, and the copies zero-fill the columns beyond a head size.
 #include "common.cuh"
 #include "kernels.h"
 #include "launch.cuh"
+#include "stack.h"
 
 namespace cb {
 
@@ -77,21 +82,47 @@ __device__ __forceinline__ float pt_ex2(float x) {
   return y;
 }
 
-__device__ __forceinline__ void pt_bar_sync() { asm volatile("bar.sync 1, 128;" ::: "memory"); }
+// Barrier of the 128 softmax threads that also tells each of them whether any has given up on a wait: a thread whose
+// wait expired keeps coming to the barriers until all leave together, so that none is left waiting for it.
+__device__ __forceinline__ bool pt_bar_all_ok(bool ok) {
+  int bad;
+  asm volatile(
+      "{\n\t.reg .pred p, r;\n\t"
+      "setp.ne.b32 p, %1, 0;\n\t"
+      "barrier.red.or.pred r, 1, 128, p;\n\t"
+      "selp.b32 %0, 1, 0, r;\n\t}"
+      : "=r"(bad)
+      : "r"(ok ? 0 : 1)
+      : "memory");
+  return bad == 0;
+}
 
-struct PtItem {
-  int split, kvh, b, kv_begin, kv_end, n_tiles;
+// Window, bias and layout of a WIN launch (the plain kernel has no window, no bias and packed 128-wide heads).
+struct PtWin {
+  int window, kdim, vdim;
+  const float* r1;   // [Hq]; null = no bias
+  const float* r2;
+  long long ldq, ldo;
 };
 
-__device__ __forceinline__ PtItem pt_item(int it, int n_splits, int Hkv, const int* __restrict__ seq_lens) {
+struct PtItem {
+  int split, kvh, b, len, kv_begin, kv_end, n_tiles;
+};
+
+template <bool WIN>
+__device__ __forceinline__ PtItem pt_item(int it, int n_splits, int Hkv, const int* __restrict__ seq_lens, const PtWin& w,
+                                          int page_size) {
   PtItem I;
   I.split = it % n_splits;
   I.kvh = (it / n_splits) % Hkv;
   I.b = it / (n_splits * Hkv);
-  const int len = seq_lens[I.b];
-  const int chunk = ((len + n_splits - 1) / n_splits + PT_TILE - 1) / PT_TILE * PT_TILE;
-  I.kv_begin = I.split * chunk;
-  I.kv_end = min(len, I.kv_begin + chunk);
+  I.len = seq_lens[I.b];
+  // first token read: the start of the page that holds the oldest visible key
+  const int first = WIN ? max(0, I.len - w.window) / page_size * page_size : 0;
+  const int span = I.len - first;
+  const int chunk = ((span + n_splits - 1) / n_splits + PT_TILE - 1) / PT_TILE * PT_TILE;
+  I.kv_begin = first + I.split * chunk;
+  I.kv_end = min(I.len, I.kv_begin + chunk);
   I.n_tiles = I.kv_end > I.kv_begin ? (I.kv_end - I.kv_begin + PT_TILE - 1) / PT_TILE : 0;
   return I;
 }
@@ -99,13 +130,13 @@ __device__ __forceinline__ PtItem pt_item(int it, int n_splits, int Hkv, const i
 // Persistent: CTA c works on items c, c + gridDim.x, ... (item = one (sequence, kv head, kv split)); the
 // K/V ring, the barriers and the global tile counter `gt` run on across items, so the copies of the
 // next item's first tiles are in flight while the current item finishes.
-template <int GROUP>
+template <int GROUP, bool WIN>
 __global__ void __launch_bounds__(PT_THREADS, 1)
 paged_decode_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV,
                        const bf16* __restrict__ q, const int* __restrict__ table, const int* __restrict__ seq_lens,
                        int max_pages, int page_size, int num_pages, int n_seqs, int Hq, int Hkv, int n_splits,
                        float scale_log2, float* __restrict__ part_acc, float* __restrict__ part_ml,
-                       bf16* __restrict__ out, int* __restrict__ status) {
+                       bf16* __restrict__ out, int* __restrict__ status, const PtWin win) {
   extern __shared__ uint8_t smem_raw[];
   const uint32_t base = (smem_u32(smem_raw) + 1023u) & ~1023u;
   uint8_t* gen = smem_raw + (base - smem_u32(smem_raw));
@@ -126,6 +157,9 @@ paged_decode_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_con
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int n_items = n_splits * Hkv * n_seqs;
+  // 64-column halves that hold data, and 16-column steps of the first product
+  const int k_halves = WIN && win.kdim <= 64 ? 1 : 2, v_halves = WIN && win.vdim <= 64 ? 1 : 2;
+  const int k_steps = WIN ? (win.kdim + 15) / 16 : 8;
 
   // ---- setup: barriers, TMEM, operand buffers zeroed (rows >= GROUP of Q^T / P^T stay zero for good)
   if (threadIdx.x == 0) {
@@ -171,7 +205,7 @@ paged_decode_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_con
     bool ok = true;
     int issued_lo = 0;
     for (int it = blockIdx.x; it < n_items && ok; it += gridDim.x) {
-      const PtItem I = pt_item(it, n_splits, Hkv, seq_lens);
+      const PtItem I = pt_item<WIN>(it, n_splits, Hkv, seq_lens, win, page_size);
       if (I.n_tiles == 0) continue;
       // Q^T buffer of this item: a ring of PT_NQ. It is written below after the wait for the ring slot of
       // the item's first tile T0, which returns once tile T0 - PT_NST has been consumed; the previous user of
@@ -212,19 +246,22 @@ paged_decode_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_con
         if (j == 0) {
           for (int i = lane; i < GROUP * 128; i += 32) {
             const int g = i >> 7, d = i & 127;
+            if (WIN && d >= win.kdim) continue;   // those columns stay zero
             *reinterpret_cast<bf16*>(opb_gen + PT_OPB * qb + opb_offset(g, d)) =
-                q[((long long)I.b * Hq + I.kvh * GROUP + g) * 128 + d];
+                WIN ? q[(long long)I.b * win.ldq + (long long)(I.kvh * GROUP + g) * win.kdim + d]
+                    : q[((long long)I.b * Hq + I.kvh * GROUP + g) * 128 + d];
           }
           fence_proxy_async();
         }
         __syncwarp();
-        if (lane == 0) mbar_arrive_expect_tx(full, 2 * PT_TILE_BYTES);
+        if (lane == 0) mbar_arrive_expect_tx(full, WIN ? (k_halves + v_halves) * PT_HALF : 2 * PT_TILE_BYTES);
         __syncwarp();
 #pragma unroll
         for (int r = 0; r < 2; ++r) {
           const int op = lane + 32 * r;
           if (op < n_ops) {
             const int which = op & 3;
+            if (WIN && (which & 1) && ((which & 2) ? v_halves : k_halves) == 1) continue;
             const uint32_t dst = ((which & 2) ? v_smem(s) : k_smem(s)) + ((which & 1) ? PT_HALF : 0) +
                                  uint32_t((op >> 2) * page_size) * 128u;
             tma_load_4d(dst, (which & 2) ? &tmV : &tmK, full, (which & 1) ? 64 : 0, 0, I.kvh, r ? cur1 : cur0);
@@ -247,7 +284,7 @@ paged_decode_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_con
     int gt = 0, io = 0;
     bool ok = true;
     for (int it = blockIdx.x; it < n_items && ok; it += gridDim.x) {
-      const PtItem I = pt_item(it, n_splits, Hkv, seq_lens);
+      const PtItem I = pt_item<WIN>(it, n_splits, Hkv, seq_lens, win, page_size);
       if (I.n_tiles == 0) continue;
       const uint64_t q_desc = make_smem_desc_sw128(q_smem(io % PT_NQ), 16, 1024);
       auto issue_s = [&](int g) {
@@ -255,6 +292,7 @@ paged_decode_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_con
         const uint32_t d = T_S0 + 16 * (g & 1);
 #pragma unroll
         for (int kk = 0; kk < 8; ++kk) {
+          if (WIN && kk >= k_steps) break;
           const uint32_t ka = (kk >> 2) * (PT_HALF >> 4) + 2 * (kk & 3);
           const uint32_t kb = (kk >> 2) * (2048 >> 4) + 2 * (kk & 3);
           mma_ss(d, k_desc + ka, q_desc + kb, idesc_s, kk > 0 ? 1u : 0u);
@@ -296,33 +334,40 @@ paged_decode_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_con
     const int t = quad * 32 + lane;
     const uint32_t lane_addr = uint32_t(quad * 32) << 16;
     int gt = 0;
-    bool ok = true;
-    for (int it = blockIdx.x; it < n_items && ok; it += gridDim.x) {
-      const PtItem I = pt_item(it, n_splits, Hkv, seq_lens);
-      float m_used[GROUP], l_part[GROUP];
+    bool ok = true, left = false;   // left: all 128 threads have agreed to stop
+    for (int it = blockIdx.x; it < n_items && !left; it += gridDim.x) {
+      const PtItem I = pt_item<WIN>(it, n_splits, Hkv, seq_lens, win, page_size);
+      float m_used[GROUP], l_part[GROUP], b1[GROUP], b2[GROUP];
 #pragma unroll
-      for (int g = 0; g < GROUP; ++g) { m_used[g] = -1e30f; l_part[g] = 0.f; }
+      for (int g = 0; g < GROUP; ++g) {
+        m_used[g] = -1e30f; l_part[g] = 0.f;
+        b1[g] = WIN && win.r1 ? win.r1[I.kvh * GROUP + g] : 0.f;
+        b2[g] = WIN && win.r1 ? win.r2[I.kvh * GROUP + g] : 0.f;
+      }
       for (int j = 0; j < I.n_tiles; ++j, ++gt) {
-        if (!mbar_wait(B(PB_S + (gt & 1)), (gt >> 1) & 1, abort_flag, status, ST_TIMEOUT_SOFTMAX)) {
-          ok = false;
-          break;
-        }
+        ok = ok && mbar_wait(B(PB_S + (gt & 1)), (gt >> 1) & 1, abort_flag, status, ST_TIMEOUT_SOFTMAX);
+        __syncwarp();
         tc_fence_after();
         uint32_t sv[16];
         tmem_ld16(T_S0 + 16 * (gt & 1) + lane_addr, sv);
         tmem_wait_ld();
-        const bool valid = I.kv_begin + j * PT_TILE + t < I.kv_end;
+        const int pos = I.kv_begin + j * PT_TILE + t;
+        const int dist = I.len - 1 - pos;
+        const bool valid = pos < I.kv_end && (!WIN || dist < win.window);
         float x[GROUP], tm[GROUP];
         float* rbuf = red + (gt & 1) * 4 * GROUP;
 #pragma unroll
         for (int g = 0; g < GROUP; ++g) {
-          x[g] = valid ? __uint_as_float(sv[g]) * scale_log2 : -1e30f;
+          x[g] = __uint_as_float(sv[g]) * scale_log2;
+          if (WIN) x[g] -= b1[g] * __log2f(fmaf(b2[g], (float)dist, 1.f));
+          x[g] = valid ? x[g] : -1e30f;
           float v = x[g];
 #pragma unroll
           for (int o = 16; o > 0; o >>= 1) v = fmaxf(v, __shfl_xor_sync(0xffffffffu, v, o));
           if (lane == 0) rbuf[quad * GROUP + g] = v;
         }
-        pt_bar_sync();
+        left = !pt_bar_all_ok(ok);
+        if (left) break;
         bool need = false;
 #pragma unroll
         for (int g = 0; g < GROUP; ++g) {
@@ -335,10 +380,8 @@ paged_decode_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_con
           for (int g = 0; g < GROUP; ++g) m_used[g] = tm[g];
         } else if (need) {
           // the running max moved by more than 2^8 for some head: rescale O^T once every earlier product is done
-          if (!mbar_wait(B(PB_PV + ((gt - 1) & 1)), ((gt - 1) >> 1) & 1, abort_flag, status, ST_TIMEOUT_SOFTMAX)) {
-            ok = false;
-            break;
-          }
+          ok = mbar_wait(B(PB_PV + ((gt - 1) & 1)), ((gt - 1) >> 1) & 1, abort_flag, status, ST_TIMEOUT_SOFTMAX);
+          __syncwarp();
           tc_fence_after();
           uint32_t ov[16];
           tmem_ld16(T_O + lane_addr, ov);
@@ -357,10 +400,7 @@ paged_decode_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_con
           tc_fence_before();
         }
         // P buffer (gt & 1) was last read by the second product of global tile gt - 2
-        if (gt >= 2 && !mbar_wait(B(PB_PV + (gt & 1)), ((gt >> 1) - 1) & 1, abort_flag, status, ST_TIMEOUT_SOFTMAX)) {
-          ok = false;
-          break;
-        }
+        if (gt >= 2 && ok) ok = mbar_wait(B(PB_PV + (gt & 1)), ((gt >> 1) - 1) & 1, abort_flag, status, ST_TIMEOUT_SOFTMAX);
         uint8_t* pbuf = opb_gen + PT_OPB * (PT_NQ + (gt & 1));
 #pragma unroll
         for (int g = 0; g < GROUP; ++g) {
@@ -371,7 +411,7 @@ paged_decode_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_con
         fence_proxy_async();
         mbar_arrive(B(PB_P + (gt & 1)));
       }
-      if (!ok) break;
+      if (left) break;
       // ---- item epilogue: row sums over the 128 threads, then this thread's output dim for every head
       uint32_t ov[16];
 #pragma unroll
@@ -388,13 +428,12 @@ paged_decode_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_con
           for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
           if (lane == 0) rbuf[quad * GROUP + g] = v;
         }
-        pt_bar_sync();
+        left = !pt_bar_all_ok(ok);
+        if (left) break;
 #pragma unroll
         for (int g = 0; g < GROUP; ++g) l[g] = rbuf[g] + rbuf[GROUP + g] + rbuf[2 * GROUP + g] + rbuf[3 * GROUP + g];
-        if (!mbar_wait(B(PB_PV + ((gt - 1) & 1)), ((gt - 1) >> 1) & 1, abort_flag, status, ST_TIMEOUT_SOFTMAX)) {
-          ok = false;
-          break;
-        }
+        ok = mbar_wait(B(PB_PV + ((gt - 1) & 1)), ((gt - 1) >> 1) & 1, abort_flag, status, ST_TIMEOUT_SOFTMAX);
+        __syncwarp();
         tc_fence_after();
         tmem_ld16(T_O + lane_addr, ov);
         tmem_wait_ld();
@@ -405,7 +444,11 @@ paged_decode_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_con
         const int h = I.kvh * GROUP + g;
         const float a = __uint_as_float(ov[g]);
         if (n_splits == 1) {
-          out[((long long)I.b * Hq + h) * 128 + t] = __float2bfloat16(l[g] > 0.f ? a / l[g] : 0.f);
+          const bf16 o = __float2bfloat16(l[g] > 0.f ? a / l[g] : 0.f);
+          if (!WIN)
+            out[((long long)I.b * Hq + h) * 128 + t] = o;
+          else if (t < win.vdim)
+            out[(long long)I.b * win.ldo + (long long)h * win.vdim + t] = o;
         } else {
           const long long pb = ((long long)I.b * Hq + h) * n_splits + I.split;
           part_acc[pb * 128 + t] = a;
@@ -425,6 +468,23 @@ paged_decode_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_con
     tc_fence_after();
     tmem_dealloc(tmem_base, 64);
   }
+}
+
+// Merge of a WIN launch's splits (partial rows of 128): out[b, h, d] with the launch's output layout.
+__global__ void __launch_bounds__(128)
+window_decode_merge_kernel(const float* __restrict__ part_acc, const float* __restrict__ part_ml, int n_splits, int Hq,
+                           int vdim, long long ldo, bf16* __restrict__ out) {
+  const long long bh = blockIdx.x;
+  const int d = threadIdx.x;
+  float m = -1e30f;
+  for (int s = 0; s < n_splits; ++s) m = fmaxf(m, part_ml[(bh * n_splits + s) * 2]);
+  float num = 0.f, den = 0.f;
+  for (int s = 0; s < n_splits; ++s) {
+    const float w = exp2f(part_ml[(bh * n_splits + s) * 2] - m);
+    num += w * part_acc[(bh * n_splits + s) * 128 + d];
+    den += w * part_ml[(bh * n_splits + s) * 2 + 1];
+  }
+  if (d < vdim) out[bh / Hq * ldo + bh % Hq * vdim + d] = __float2bfloat16(den > 0.f ? num / den : 0.f);
 }
 
 }  // namespace cb
@@ -457,22 +517,23 @@ bool paged_decode_tc_supported(const PagedDecodeArgs& a) {
          (ps == 8 || ps == 16 || ps == 32 || ps == 64 || ps == 128);
 }
 
-static CUtensorMap cache_map(const void* base, int num_pages, int Hkv, int page_size) {
-  const uint64_t dims[4] = {128, (uint64_t)page_size, (uint64_t)Hkv, (uint64_t)num_pages};
-  const uint64_t strides[3] = {256, (uint64_t)page_size * 256, (uint64_t)Hkv * page_size * 256};
+static CUtensorMap cache_map(const void* base, int num_pages, int Hkv, int page_size, int dim = 128) {
+  const uint64_t dims[4] = {(uint64_t)dim, (uint64_t)page_size, (uint64_t)Hkv, (uint64_t)num_pages};
+  const uint64_t row = (uint64_t)dim * 2;
+  const uint64_t strides[3] = {row, (uint64_t)page_size * row, (uint64_t)Hkv * page_size * row};
   const uint32_t box[4] = {64, (uint32_t)page_size, 1, 1};
   return cbh::make_tmap_bf16(base, 4, dims, strides, box, true);
 }
 
-template <int GROUP>
-static void launch_tc(const PagedDecodeArgs& a, float* pa, float* pm, cudaStream_t s) {
+template <int GROUP, bool WIN>
+static void launch_tc(const PagedDecodeArgs& a, const cb::PtWin& w, float* pa, float* pm, cudaStream_t s) {
   static thread_local bool configured = false;
   if (!configured) {
-    cudaFuncSetAttribute(cb::paged_decode_tc_kernel<GROUP>, cudaFuncAttributeMaxDynamicSharedMemorySize, cb::PT_SMEM);
+    cudaFuncSetAttribute(cb::paged_decode_tc_kernel<GROUP, WIN>, cudaFuncAttributeMaxDynamicSharedMemorySize, cb::PT_SMEM);
     configured = true;
   }
-  CUtensorMap tk = cache_map(a.k_cache, a.num_pages, a.Hkv, a.page_size);
-  CUtensorMap tv = cache_map(a.v_cache, a.num_pages, a.Hkv, a.page_size);
+  CUtensorMap tk = cache_map(a.k_cache, a.num_pages, a.Hkv, a.page_size, w.kdim);
+  CUtensorMap tv = cache_map(a.v_cache, a.num_pages, a.Hkv, a.page_size, w.vdim);
   // persistent: one CTA per SM walks over the (sequence, kv head, split) items
   static thread_local int sms = 0;
   if (sms == 0) {
@@ -483,23 +544,58 @@ static void launch_tc(const PagedDecodeArgs& a, float* pa, float* pm, cudaStream
   }
   const long long items = (long long)a.n_splits * a.Hkv * a.B;
   const int grid = (int)std::min<long long>(items, sms);
-  launch_pdl(cb::paged_decode_tc_kernel<GROUP>, dim3(grid), dim3(cb::PT_THREADS), cb::PT_SMEM, s,
+  launch_pdl(cb::paged_decode_tc_kernel<GROUP, WIN>, dim3(grid), dim3(cb::PT_THREADS), cb::PT_SMEM, s,
       tk, tv, (const bf16*)a.q, a.block_table, a.seq_lens, a.max_pages, a.page_size, a.num_pages, a.B, a.Hq, a.Hkv,
-      a.n_splits, a.scale * 1.4426950408889634f, pa, pm, (bf16*)a.out, a.status);
+      a.n_splits, a.scale * 1.4426950408889634f, pa, pm, (bf16*)a.out, a.status, w);
 }
 
 // Launches the tensor-core kernel (partials into pa / pm when n_splits > 1; the caller merges them: a merge by the
 // CTA that finishes a head's last split was measured slower, 12.81 against 12.45 ms per decode step at batch 32,
 // because every item then pays a device-scope fence on the softmax threads' path).
 // The caller has checked paged_decode_tc_supported().
-void paged_decode_tc_launch(const PagedDecodeArgs& a, float* pa, float* pm, cudaStream_t s) {
+template <bool WIN>
+static void launch_group(const PagedDecodeArgs& a, const cb::PtWin& w, float* pa, float* pm, cudaStream_t s) {
   switch (a.Hq / a.Hkv) {
-    case 1: launch_tc<1>(a, pa, pm, s); break;
-    case 2: launch_tc<2>(a, pa, pm, s); break;
-    case 4: launch_tc<4>(a, pa, pm, s); break;
-    case 8: launch_tc<8>(a, pa, pm, s); break;
+    case 1: launch_tc<1, WIN>(a, w, pa, pm, s); break;
+    case 2: launch_tc<2, WIN>(a, w, pa, pm, s); break;
+    case 4: launch_tc<4, WIN>(a, w, pa, pm, s); break;
+    case 8: launch_tc<8, WIN>(a, w, pa, pm, s); break;
     default: throw std::runtime_error("paged_decode_tc: Hq / Hkv must be 1, 2, 4 or 8");
   }
+}
+void paged_decode_tc_launch(const PagedDecodeArgs& a, float* pa, float* pm, cudaStream_t s) {
+  launch_group<false>(a, cb::PtWin{0, 128, 128, nullptr, nullptr, 0, 0}, pa, pm, s);
+}
+
+// ---- decode steps of windowed attention (stack.h)
+static PagedDecodeArgs paged_args(const WindowAttnArgs& a) {
+  PagedDecodeArgs d;
+  d.q = a.q; d.k_cache = a.k_cache; d.v_cache = a.v_cache; d.block_table = a.table; d.seq_lens = a.seq_lens; d.out = a.out;
+  d.B = a.n_seqs; d.Hq = a.H; d.Hkv = a.G; d.page_size = a.page_size; d.max_pages = a.max_pages; d.num_pages = a.num_pages;
+  d.scale = a.scale; d.n_splits = a.n_splits; d.status = a.status;
+  return d;
+}
+
+bool window_attn_decode_tc_supported(const WindowAttnArgs& a) {
+  return window_attn_tc_supported(a) && paged_decode_tc_supported(paged_args(a));
+}
+
+int window_attn_decode_splits(int n_seqs, int G, int span) { return paged_decode_tc_pick_splits(n_seqs, G, span); }
+
+size_t window_attn_scratch_bytes(int n_seqs, int H, int vdim, int n_splits) {
+  (void)vdim;   // partial rows are 128 wide whatever the head size
+  return n_splits <= 1 ? 0 : (size_t)n_seqs * H * n_splits * (128 + 2) * sizeof(float);
+}
+
+void window_attn_decode_tc(const WindowAttnArgs& a, cudaStream_t s) {
+  if (a.n_seqs <= 0) return;
+  if (a.n_splits < 1 || a.n_splits > 64 || a.window < 1 || a.scratch_bytes < window_attn_scratch_bytes(a.n_seqs, a.H, a.vdim, a.n_splits))
+    throw std::runtime_error("window_attn_decode_tc: bad split count or scratch buffer");
+  float* pa = a.n_splits > 1 ? a.scratch : nullptr;
+  float* pm = pa ? pa + (size_t)a.n_seqs * a.H * a.n_splits * 128 : nullptr;
+  launch_group<true>(paged_args(a), cb::PtWin{a.window, a.dim, a.vdim, a.r1, a.r2, a.ldq, a.ldo}, pa, pm, s);
+  if (pa)
+    cb::window_decode_merge_kernel<<<a.n_seqs * a.H, 128, 0, s>>>(pa, pm, a.n_splits, a.H, a.vdim, a.ldo, (bf16*)a.out);
 }
 
 }  // namespace cosmos
