@@ -124,7 +124,11 @@ class StackModel(nn.Module):
     def load(self, model_dir) -> "StackModel":
         from ..ckpt import safetensors_io as sio
 
-        sio.load_into(model_dir, {k: v.data for k, v in self.checkpoint_views().items()})
+        targets = {k: v.data for k, v in self.checkpoint_views().items()}
+        unused = f"l{self.first_mix}.mix.vmix"   # the first mixing layer has nothing to mix with
+        if unused in targets and unused not in sio.tensor_files(model_dir):
+            del targets[unused]
+        sio.load_into(model_dir, targets)
         return self.check_tables()
 
     def check_tables(self) -> "StackModel":

@@ -35,7 +35,7 @@ def build_parser() -> argparse.ArgumentParser:
                                  formatter_class=argparse.RawDescriptionHelpFormatter)
     ap.add_argument("-i", "--input", required=True, help="input spec: .json (one sample) or .jsonl (one per line)")
     ap.add_argument("-o", "--output", required=True, help="output root; one sub-directory per sample name")
-    ap.add_argument("--checkpoint-path", default="Cosmos3-Nano", help="model name (resolved under nvidia/) or path")
+    ap.add_argument("--checkpoint-path", default="Cosmos3-Nano", help="model name (resolved under nvidia/) or path; a decoder stack by registered name or directory")
     ap.add_argument("--parallelism-preset", choices=["latency", "throughput"], default=None)
     ap.add_argument("--dp-shard-size", type=int, default=None)
     ap.add_argument("--dp-replicate-size", type=int, default=None)
@@ -221,7 +221,7 @@ def _reasoner_prompt(tokenizer, vit, cfg, spec: InferenceSpec, device):
 
 def run_reasoner_batch(pipe, vit, specs: List[InferenceSpec], out_root: Path, is_writer: bool, device,
                        max_num_seqs: int = 32) -> List[Dict]:
-    """All reasoner samples of a spec file through the continuous-batching engine (`serve/engine.py`): they
+    """All reasoner samples of a spec file (any model that `serve/engine.py` serves) through the continuous-batching engine (`serve/engine.py`): they
     share decode steps (one CUDA graph per step on a GPU), each with its own sampling parameters."""
     from ..models.reasoner import ReasonerEngine
     from ..serve.engine import BatchEngine
@@ -257,6 +257,38 @@ def run_reasoner_batch(pipe, vit, specs: List[InferenceSpec], out_root: Path, is
                         "tokens_per_s": len(r.out) / dt, "prompt_tokens": len(r.ids), "completion_tokens": len(r.out),
                         "batch_wall_s": wall, "batch_tokens_per_s": sum(len(q.out) for q in reqs) / max(wall, 1e-9)})
     return records
+
+
+def run_stack(args, specs: List[InferenceSpec]) -> int:
+    """Reasoner-mode samples of a decoder stack (a checkpoint directory whose config.json names its architecture, or a
+    registered name): token prompts through the batching engine, on one GPU."""
+    from types import SimpleNamespace
+
+    from ..models.stack import load_stack
+    from ..utils.tokenizer import load_tokenizer
+
+    bad = [s.name for s in specs if s.model_mode != "reasoner" or s.vision_path]
+    if bad:
+        print(f"spec error: {args.checkpoint_path} generates text from text only (sample {bad[0]})", file=sys.stderr)
+        return 2
+    if int(os.environ.get("WORLD_SIZE", "1")) > 1:
+        print("parallelism error: decoder stacks run on one GPU", file=sys.stderr)
+        return 2
+    use_cuda = torch.cuda.is_available() and args.device != "cpu"
+    device = torch.device("cuda", 0) if use_cuda else torch.device("cpu")
+    dtype = torch.bfloat16 if (args.dtype or ("bf16" if use_cuda else "fp32")) == "bf16" else torch.float32
+    model = load_stack(args.checkpoint_path, dtype, device)
+    ckpt = args.checkpoint_path if Path(args.checkpoint_path).is_dir() else None
+    pipe = SimpleNamespace(transformer=model, cfg=model.cfg, device=device, tokenizer=load_tokenizer(ckpt, model.cfg.vocab_size))
+    out_root = Path(args.output)
+    out_root.mkdir(parents=True, exist_ok=True)
+    records = run_reasoner_batch(pipe, None, specs, out_root, True, device)
+    for rec in records:
+        print(json.dumps(rec), flush=True)
+    if args.benchmark:
+        avg = {k: sum(r[k] for r in records) / len(records) for k in ("generation_time_s", "tokens_per_s")}
+        (out_root / "benchmark.json").write_text(json.dumps({"average": avg, "samples": records, "world_size": 1}, indent=1))
+    return 0
 
 
 def run_reasoner_sample(engine, tokenizer, vit, spec: InferenceSpec, out_dir: Path, is_writer: bool, device) -> Dict:
@@ -305,6 +337,9 @@ def main(argv: Optional[List[str]] = None) -> int:
     except SpecError as e:
         print(f"spec error: {e}", file=sys.stderr)
         return 2
+    from ..models.stack import is_stack_name
+    if is_stack_name(args.checkpoint_path):
+        return run_stack(args, specs)
     world = int(os.environ.get("WORLD_SIZE", "1"))
     rank = int(os.environ.get("RANK", "0"))
     local_rank = int(os.environ.get("LOCAL_RANK", "0"))

@@ -359,7 +359,7 @@ class Cosmos3Server:
         return out
 
     def _chat_completions(self, body: dict, on_token=None) -> dict:
-        if self.reasoner is None:
+        if self.reasoner is None and self.batch_engine is None:
             raise RuntimeError("this server was started without the Reasoner")
         t0 = time.time()
         tok = self.pipe.tokenizer
@@ -376,6 +376,8 @@ class Cosmos3Server:
                 parts = []
                 for part in content:
                     kind = part.get("type")
+                    if kind in ("image_url", "video_url") and self.vit is None:
+                        raise ValueError("this model takes text only")
                     if kind in ("image_url", "video_url"):
                         frames, times = self._load_media(part[kind]["url"], kind == "video_url", extra)
                         emb, grid, ds = self._encode_vision(frames, dev, (extra.get("mm_processor_kwargs") or {}).get("size"))
@@ -415,7 +417,7 @@ class Cosmos3Server:
         pad_id = tok.video_pad_id if has_video else tok.image_pad_id
         if ve is not None and len({tok.image_pad_id, tok.video_pad_id}) == 2:
             ids = [pad_id if t in (tok.image_pad_id, tok.video_pad_id) else t for t in ids]
-        if self.batch_engine is not None and dc.seed is None:
+        if self.batch_engine is not None and (dc.seed is None or self.reasoner is None):
             # joins the running decode batch instead of taking the generation lock (sampling runs on the
             # device; a request that pins a seed takes the single-request path). A prompt with media is
             # prefilled on its own (vision rows spliced in, 3-D rotary ids, DeepStack features) and then decodes
@@ -645,6 +647,25 @@ def apply_deploy_config(args) -> None:
             args.model_class_name = stage["model_class_name"]
 
 
+def stack_server(args, device, dtype) -> Cosmos3Server:
+    """Server of a decoder stack (models/stack.py): chat completions through the batching engine; a seed in a request is
+    ignored there, and the image and video endpoints answer with an error."""
+    from types import SimpleNamespace
+
+    from ..models.stack import load_stack
+    from ..utils.tokenizer import load_tokenizer
+    from .engine import BatchEngine, EngineWorker
+
+    if args.max_num_seqs <= 0:
+        raise SystemExit("a decoder stack is served by the batching engine: --max-num-seqs must be > 0")
+    model = load_stack(args.model, dtype, device or "cpu")
+    ckpt = args.model if Path(args.model).is_dir() else None
+    pipe = SimpleNamespace(transformer=model, cfg=model.cfg, device=model.device, safety_checker=None,
+                           tokenizer=load_tokenizer(ckpt, model.cfg.vocab_size))
+    worker = EngineWorker(BatchEngine(model, max_batch=args.max_num_seqs, max_len=args.max_model_len))
+    return Cosmos3Server(pipe, None, None, args.model, False, "", batch_engine=worker)
+
+
 def main(argv=None) -> int:
     import argparse
 
@@ -692,6 +713,11 @@ def main(argv=None) -> int:
         torch.cuda.set_device(int(os.environ.get("LOCAL_RANK", "0")))
     dev = f"cuda:{int(os.environ.get('LOCAL_RANK', '0'))}" if torch.cuda.is_available() else None
     dtype = torch.bfloat16 if (dev and args.dtype == "bf16") else torch.float32
+    from ..models.stack import is_stack_name
+    if is_stack_name(args.model):
+        server = stack_server(args, dev, dtype)
+        uvicorn.run(create_app(server), host=args.host, port=args.port, log_level="info")
+        return 0
     over = json.loads(args.hf_overrides) if args.hf_overrides else {}
     reasoner_only = "Cosmos3ReasonerForConditionalGeneration" in (over.get("architectures") or [])
     pipe = Cosmos3OmniPipeline.from_pretrained(args.model, torch_dtype=dtype, device_map=dev,
