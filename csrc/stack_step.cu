@@ -48,10 +48,135 @@ template <> struct Vec<bf16, 4> {
   }
 };
 
+template <> struct Vec<float, 8> {
+  static __device__ __forceinline__ void load(const float* p, float (&v)[8]) {
+    const float4 x = reinterpret_cast<const float4*>(p)[0], y = reinterpret_cast<const float4*>(p)[1];
+    v[0] = x.x; v[1] = x.y; v[2] = x.z; v[3] = x.w; v[4] = y.x; v[5] = y.y; v[6] = y.z; v[7] = y.w;
+  }
+  static __device__ __forceinline__ void store(float* p, const float (&v)[8]) {
+    reinterpret_cast<float4*>(p)[0] = make_float4(v[0], v[1], v[2], v[3]);
+    reinterpret_cast<float4*>(p)[1] = make_float4(v[4], v[5], v[6], v[7]);
+  }
+};
+template <> struct Vec<bf16, 8> {
+  static __device__ __forceinline__ void load(const bf16* p, float (&v)[8]) {
+    const uint4 x = *reinterpret_cast<const uint4*>(p);
+    v[0] = bf16lo(x.x); v[1] = bf16hi(x.x); v[2] = bf16lo(x.y); v[3] = bf16hi(x.y);
+    v[4] = bf16lo(x.z); v[5] = bf16hi(x.z); v[6] = bf16lo(x.w); v[7] = bf16hi(x.w);
+  }
+  static __device__ __forceinline__ void store(bf16* p, const float (&v)[8]) {
+    uint4 o;
+    o.x = pack_bf16(v[0], v[1]); o.y = pack_bf16(v[2], v[3]); o.z = pack_bf16(v[4], v[5]); o.w = pack_bf16(v[6], v[7]);
+    *reinterpret_cast<uint4*>(p) = o;
+  }
+};
+
 __device__ __forceinline__ float warp_add(float v) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
   return v;
+}
+
+// The common case of residual_norm_kernel (below), tuned for whole prompts: at most 4 vectors of 8 per thread, kept in
+// registers (all loads of a row are issued before the first use), one or two parts of at least a warp's vectors each.
+template <typename T, typename Y, int NV>
+__global__ void __launch_bounds__(256)
+residual_norm_row_kernel(const cosmos::ResidualNormArgs a) {
+  __shared__ float part_s[2][8];
+  const long long r = blockIdx.x;
+  const int tid = threadIdx.x, nt = blockDim.x, warp = tid >> 5, lane = tid & 31, warps = nt >> 5;
+  const int d = a.d;
+  float* xr = a.x + r * d;
+  float v[NV][8];
+  if (a.embed) {
+    long long tok = a.tokens[r];
+    if (!index_ok(tok, a.vocab, a.status, SITE_STACK_TOKEN)) tok = 0;
+    const T* er = reinterpret_cast<const T*>(a.embed) + tok * a.ld_embed;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = (tid + i * nt) * 8;
+      if (c < d) {
+        Vec<T, 8>::load(er + c, v[i]);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) v[i][e] *= a.embed_scale;
+      }
+    }
+  } else {
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = (tid + i * nt) * 8;
+      if (c < d) Vec<float, 8>::load(xr + c, v[i]);
+    }
+  }
+  if (a.y) {
+    for (int k = 0; k < a.top; ++k) {
+      const long long yr = a.y_rows ? (long long)a.y_rows[r * a.top + k] : r;
+      if (!index_ok(yr, a.y_n, a.status, SITE_MOE_ROW)) continue;
+      const Y* src = reinterpret_cast<const Y*>(a.y) + yr * a.ldy;
+      for (int ks = 0; ks < a.k_splits; ++ks, src += a.split_stride) {
+#pragma unroll
+        for (int i = 0; i < NV; ++i) {
+          const int c = (tid + i * nt) * 8;
+          if (c < d) {
+            float t[8];
+            Vec<Y, 8>::load(src + c, t);
+#pragma unroll
+            for (int e = 0; e < 8; ++e) v[i][e] = fmaf(a.weight, t[e], v[i][e]);
+          }
+        }
+      }
+    }
+  }
+  const int psize = d / a.groups;   // one or two parts
+  float ss[2] = {0.f, 0.f};
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = (tid + i * nt) * 8;
+    if (c < d) {
+      Vec<float, 8>::store(xr + c, v[i]);
+      float s = 0.f;
+#pragma unroll
+      for (int e = 0; e < 8; ++e) s = fmaf(v[i][e], v[i][e], s);
+      if (c < psize) ss[0] += s; else ss[1] += s;
+    }
+  }
+  if (!a.h) return;
+  ss[0] = warp_add(ss[0]);
+  ss[1] = warp_add(ss[1]);
+  if (lane == 0) {
+    part_s[0][warp] = ss[0];
+    part_s[1][warp] = ss[1];
+  }
+  __syncthreads();
+  float rinv[2] = {0.f, 0.f};
+  for (int w = 0; w < warps; ++w) {
+    rinv[0] += part_s[0][w];
+    rinv[1] += part_s[1][w];
+  }
+  rinv[0] = 1.f / sqrtf(rinv[0] / (float)psize + a.eps);
+  rinv[1] = 1.f / sqrtf(rinv[1] / (float)psize + a.eps);
+  const T* gamma = reinterpret_cast<const T*>(a.gamma);
+  T* h = reinterpret_cast<T*>(a.h);
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = (tid + i * nt) * 8;
+    if (c < d) {
+      float g[8];
+      Vec<T, 8>::load(gamma + c, g);
+      const float q = c < psize ? rinv[0] : rinv[1];
+#pragma unroll
+      for (int e = 0; e < 8; ++e) v[i][e] = v[i][e] * q * g[e];
+    }
+  }
+  for (int k = 0; k < (a.h_rows ? a.h_top : 1); ++k) {
+    const long long hr = a.h_rows ? (long long)a.h_rows[r * a.h_top + k] : r;
+    if (!index_ok(hr, a.h_n, a.status, SITE_MOE_ROW)) continue;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = (tid + i * nt) * 8;
+      if (c < d) Vec<T, 8>::store(h + hr * a.ldh + c, v[i]);
+    }
+  }
 }
 
 // One CTA per token row; the updated row is kept in shared memory between the sum and the norm.
@@ -222,6 +347,80 @@ qkv_value_post_kernel(const cosmos::QkvValueArgs a) {
   }
 }
 
+// The same for head sizes that are multiples of 8: `lanes` threads (a power of two that covers the larger head) share a
+// head, 8 elements each, so a row moves in 16-byte pieces.
+template <typename T>
+__global__ void __launch_bounds__(256)
+qkv_value_post_vec_kernel(const cosmos::QkvValueArgs a, int lanes) {
+  const int nq = a.partial ? a.H : 0;
+  const int heads = nq + 2 * a.G;
+  const long long w = ((long long)blockIdx.x * blockDim.x + threadIdx.x) / lanes;
+  const int sub = threadIdx.x & (lanes - 1);
+  const bool live = w < a.n * heads;    // dead lanes stay for the shuffles
+  const long long t = live ? w / heads : 0;
+  const int h = live ? (int)(w - t * heads) : 0;
+  const int kind = h < nq ? 0 : (h < nq + a.G ? 1 : 2);
+  const int hh = kind == 0 ? h : (kind == 1 ? h - nq : h - nq - a.G);
+  const int size = kind == 2 ? a.vdim : a.dim;
+  const int col = kind == 0 ? hh * a.dim : (kind == 1 ? (a.H + hh) * a.dim : (a.H + a.G) * a.dim + hh * a.vdim);
+  const int c = sub * 8;
+  const bool in = live && c < size;
+  float v[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+  if (in) {
+    if (a.partial) {
+      const float* p = a.partial + t * a.ld_partial + col + c;
+#pragma unroll 4
+      for (int ks = 0; ks < a.k_splits; ++ks) {
+        float x[8];
+        Vec<float, 8>::load(p + ks * a.split_stride, x);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) v[e] += x[e];
+      }
+      if (a.bias) {
+        float x[8];
+        Vec<T, 8>::load(reinterpret_cast<const T*>(a.bias) + col + c, x);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) v[e] += x[e];
+      }
+    } else {
+      Vec<T, 8>::load(reinterpret_cast<const T*>(a.qkv) + t * a.ld + col + c, v);
+    }
+  }
+  if (kind == 2 && a.value_norm) {
+    float ss = 0.f;
+#pragma unroll
+    for (int e = 0; e < 8; ++e) ss = fmaf(v[e], v[e], ss);
+    // lanes of one head share `kind`; the mask names exactly them
+    const unsigned mask = (lanes == 32 ? 0xffffffffu : ((1u << lanes) - 1u)) << ((threadIdx.x & 31) & ~(lanes - 1));
+    for (int o = lanes >> 1; o > 0; o >>= 1) ss += __shfl_xor_sync(mask, ss, o);
+    const float rinv = 1.f / sqrtf(ss / (float)size + a.eps);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) v[e] *= rinv;
+  }
+  if (!in) return;
+  if (kind == 0) {
+    Vec<T, 8>::store(reinterpret_cast<T*>(a.q_out) + (t * a.H + hh) * a.dim + c, v);
+    return;
+  }
+  if (kind == 2) {
+    const long long fo = (t * a.G + hh) * (long long)a.vdim + c;
+    if (a.v_first_out) Vec<float, 8>::store(a.v_first_out + fo, v);
+    if (a.v_first_in) {
+      const float lam = *a.lam;
+      float f[8];
+      Vec<float, 8>::load(a.v_first_in + fo, f);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) v[e] = (1.f - lam) * v[e] + lam * f[e];
+    }
+  }
+  const long long slot = a.slots[t];
+  if (!index_ok(slot, a.n_slots, a.status, SITE_STACK_SLOT)) return;
+  const long long page = slot / a.page_size;
+  const int off = (int)(slot - page * a.page_size);
+  Vec<T, 8>::store(reinterpret_cast<T*>(kind == 1 ? a.k_cache : a.v_cache) +
+                       ((page * a.G + hh) * a.page_size + off) * (long long)size + c, v);
+}
+
 // Counting sort of the step's (token, k) pairs by expert, one CTA per layer. The order inside an expert is arbitrary:
 // the rows of a product do not depend on one another.
 __global__ void __launch_bounds__(1024)
@@ -348,6 +547,21 @@ void residual_norm(const ResidualNormArgs& a, cudaStream_t s) {
   const bool vec = psize % 4 == 0 && a.ldy % 4 == 0 && a.split_stride % 4 == 0 && a.ldh % 4 == 0 && a.ld_embed % 4 == 0 &&
                    aligned(a.x, 16) && aligned(a.y, 4 * ye) && aligned(a.h, 4 * te) && aligned(a.gamma, 4 * te) &&
                    aligned(a.embed, 4 * te);
+  // whole prompts with one or two norm parts: rows in registers
+  const bool vec8 = vec && psize % 8 == 0 && a.d % 8 == 0 && a.groups <= 2 && a.d <= 8192 && a.ldy % 8 == 0 &&
+                    a.split_stride % 8 == 0 && a.ldh % 8 == 0 && a.ld_embed % 8 == 0 && aligned(a.y, 16) && aligned(a.h, 16) &&
+                    aligned(a.gamma, 16) && aligned(a.embed, 16);
+  if (vec8 && a.rows > 296 && !a.is_f32 && !a.y_f32) {
+    const int vecs = a.d / 8;
+    const int nv = vecs <= 256 ? 1 : vecs <= 512 ? 2 : 4;
+    const int threads = std::max(32, ((vecs + nv - 1) / nv + 31) / 32 * 32);
+    switch (nv) {
+      case 1: cb::residual_norm_row_kernel<bf16, bf16, 1><<<(unsigned)a.rows, threads, 0, s>>>(a); break;
+      case 2: cb::residual_norm_row_kernel<bf16, bf16, 2><<<(unsigned)a.rows, threads, 0, s>>>(a); break;
+      default: cb::residual_norm_row_kernel<bf16, bf16, 4><<<(unsigned)a.rows, threads, 0, s>>>(a); break;
+    }
+    return;
+  }
   // few rows (a decode step): one vector per thread, so that all of a row's loads are in flight together
   const int work = (a.d + (vec ? 4 : 1) - 1) / (vec ? 4 : 1);
   const int cap = a.rows <= 296 ? 1024 : 256;
@@ -365,6 +579,19 @@ void qkv_value_post(const QkvValueArgs& a, cudaStream_t s) {
   if (a.n <= 0) return;
   if (a.dim > 512 || a.vdim > 512) throw std::runtime_error("qkv_value_post: head sizes up to 512");
   const long long warps = a.n * ((a.partial ? a.H : 0) + 2 * a.G);
+  if (a.dim % 8 == 0 && a.vdim % 8 == 0 && a.dim <= 256 && a.vdim <= 256 && a.ld % 8 == 0 && a.ld_partial % 8 == 0 &&
+      a.split_stride % 8 == 0 && aligned(a.qkv, 16) && aligned(a.partial, 16) && aligned(a.bias, 16) &&
+      aligned(a.q_out, 16) && aligned(a.k_cache, 16) && aligned(a.v_cache, 16) && aligned(a.v_first_out, 16) &&
+      aligned(a.v_first_in, 16)) {
+    int lanes = 1;
+    while (lanes * 8 < std::max(a.dim, a.vdim)) lanes *= 2;
+    const unsigned blocks = (unsigned)((warps * lanes + 255) / 256);
+    if (a.is_f32)
+      cb::qkv_value_post_vec_kernel<float><<<blocks, 256, 0, s>>>(a, lanes);
+    else
+      cb::qkv_value_post_vec_kernel<bf16><<<blocks, 256, 0, s>>>(a, lanes);
+    return;
+  }
   const unsigned grid = (unsigned)((warps + 7) / 8);
   if (a.is_f32)
     cb::qkv_value_post_kernel<float><<<grid, 256, 0, s>>>(a);

@@ -5,12 +5,15 @@
 //   * K and V come straight from the paged cache: one TMA box (page_size rows x 64 columns) per page, tensor and half, so
 //     a portion sees the tokens of earlier portions and its own through one path, and nothing is gathered beforehand.
 //   * Query tiles are listed by the host (sequence, first row, rows, position), so one launch serves portions of several
-//     sequences. Only the key blocks inside [first row's window, last row] are visited.
+//     sequences. Only the key blocks inside [first row's window, last row] are visited, and each 128-row tile skips those
+//     of them that lie outside its own rows' range.
 //   * Mask and bias are one table. Within a 128 x 128 block the distance i - j takes 255 values, so the softmax warps of a
 //     tile compute bias[i - j] once per block (two logarithms per thread), with -inf outside the window and above the
 //     diagonal, and add it with the FMA that scales the scores. A row's entries are consecutive; four copies of the table,
 //     each shifted by one entry, let every thread read four at a time with aligned 16-byte loads. The copies start 8 words
-//     apart modulo the 32 banks, so the eight lanes of a 16-byte load phase hit different banks.
+//     apart modulo the 32 banks, so the eight lanes of a 16-byte load phase hit different banks. Half of a row's entries
+//     are read before the scores are waited for (the table needs no score), which takes those loads off the chain
+//     scores -> softmax -> next product that bounds the kernel.
 //   * Head sizes up to 128 that are multiples of 8: the copies zero-fill the columns beyond the head size, products run
 //     over the 16-column steps that hold data.
 #include "common.cuh"
@@ -98,6 +101,14 @@ window_attn_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
   const int kv0 = max(0, pos0 - p.window + 1) / p.page_size * p.page_size;
   const int kv_end = pos0 + n_rows;
   const int n_blocks = (kv_end - kv0 + 127) / 128;
+  // blocks [jl, jh) of each tile: from its first row's oldest key to its last row (none for a tile without rows)
+  int jl[2], jh[2];
+#pragma unroll
+  for (int t = 0; t < 2; ++t) {
+    const int first = pos0 + t * 128, last = min(first + 127, kv_end - 1);
+    jl[t] = (max(0, first - p.window + 1) - kv0) >> 7;
+    jh[t] = last >= first ? ((last - kv0) >> 7) + 1 : jl[t];
+  }
   const int k_halves = p.kdim > 64 ? 2 : 1, v_halves = p.vdim > 64 ? 2 : 1;
 
   if (threadIdx.x == 0) {
@@ -212,10 +223,12 @@ window_attn_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
       if (ok) ok = wait_all(kv_full(0), 0);
       if (ok) {
         tc_fence_after();
-        issue_qk(0, 0);
-        commit(s_full(0));
-        issue_qk(1, 0);
-        commit(s_full(1));
+#pragma unroll
+        for (int t = 0; t < 2; ++t)
+          if (jl[t] == 0 && jh[t] > 0) {
+            issue_qk(t, 0);
+            commit(s_full(t));
+          }
         commit(kv_empty(0));
         __syncwarp();
       }
@@ -228,19 +241,21 @@ window_attn_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
         if (!ok) break;
 #pragma unroll 1
         for (int t = 0; t < 2; ++t) {
-          ok = wait_all(p_full(t, 0), j & 1);
-          if (!ok) break;
-          tc_fence_after();
-          issue_pv(t, sv, j > 0, 0);
-          ok = wait_all(p_full(t, 1), j & 1);
-          if (!ok) break;
-          tc_fence_after();
-          issue_pv(t, sv, j > 0, 1);
-          if (more) {
+          const int lo = t ? jl[1] : jl[0], hi = t ? jh[1] : jh[0];
+          if (j >= lo && j < hi) {
+            ok = wait_all(p_full(t, 0), (j - lo) & 1);
+            if (!ok) break;
+            tc_fence_after();
+            issue_pv(t, sv, j > lo, 0);
+            ok = wait_all(p_full(t, 1), (j - lo) & 1);
+            if (!ok) break;
+            tc_fence_after();
+            issue_pv(t, sv, j > lo, 1);
+            if (j + 1 == hi) commit(o_final(t));
+          }
+          if (j + 1 >= lo && j + 1 < hi) {
             issue_qk(t, sk);
             commit(s_full(t));
-          } else {
-            commit(o_final(t));
           }
           __syncwarp();
         }
@@ -266,7 +281,8 @@ window_attn_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
     float* tab_t = reinterpret_cast<float*>(gen + WA_OFF_TAB + t * 2 * WA_TAB_BYTES);
     float m_used = -1e30f, l = 0.f;
     bool ok = true;
-    for (int j = 0; j < n_blocks; ++j) {
+    const int lo = t ? jl[1] : jl[0], hi = t ? jh[1] : jh[0];
+    for (int j = lo; j < hi; ++j) {
       float* tab = tab_t + (j & 1) * (4 * WA_TAB);
       const int d0 = pos0 + t * 128 - (kv0 + j * 128);
 #pragma unroll
@@ -281,7 +297,11 @@ window_attn_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
       // the table of block j is complete; the buffer it overwrites at j + 2 has been read by every thread by then. A
       // thread that has given up on a wait keeps meeting the others here, so that nobody is left behind.
       asm volatile("bar.sync %0, 128;" ::"r"(1 + t) : "memory");
-      if (!ok || !mbar_wait(s_full(t), j & 1, abort_flag, p.status, ST_TIMEOUT_SOFTMAX)) {
+      const float4* brow = reinterpret_cast<const float4*>(tab + shift * WA_TAB + (127 - row - shift));
+      float4 bias[16];
+#pragma unroll
+      for (int c = 0; c < 16; ++c) bias[c] = brow[c];
+      if (!ok || !mbar_wait(s_full(t), (j - lo) & 1, abort_flag, p.status, ST_TIMEOUT_SOFTMAX)) {
         ok = false;
         continue;
       }
@@ -293,12 +313,11 @@ window_attn_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
       tmem_ld32(s_addr + 96, *reinterpret_cast<uint32_t(*)[32]>(&s[96]));
       tmem_wait_ld();
       // s = score * scale * log2(e) - bias, masked entries -inf; running maximum in eight chains
-      const float4* brow = reinterpret_cast<const float4*>(tab + shift * WA_TAB + (127 - row - shift));
       const uint64_t sl2_2 = wa_pack(sl2, sl2);
       float mx8[8];
 #pragma unroll
       for (int c = 0; c < 128; c += 4) {
-        const float4 b = brow[c >> 2];
+        const float4 b = c < 64 ? bias[(c >> 2) & 15] : brow[c >> 2];
         float x0, x1, x2, x3;
         wa_unpack(wa_fma2(wa_pack(__uint_as_float(s[c]), __uint_as_float(s[c + 1])), sl2_2, wa_pack(b.x, b.y)), x0, x1);
         wa_unpack(wa_fma2(wa_pack(__uint_as_float(s[c + 2]), __uint_as_float(s[c + 3])), sl2_2, wa_pack(b.z, b.w)), x2, x3);
@@ -314,7 +333,7 @@ window_attn_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
                                                              : fmaxf(mx8[e], __uint_as_float(s[i + e]));
       const float mx = wa_max3(wa_max3(mx8[0], mx8[1], mx8[2]), wa_max3(mx8[3], mx8[4], mx8[5]), fmaxf(mx8[6], mx8[7]));
       const float m_new = fmaxf(m_used, mx);
-      if (j == 0) {
+      if (j == lo) {
         m_used = m_new;
       } else {
         const bool need = m_new > m_used + 8.f;
@@ -359,8 +378,8 @@ window_attn_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
       wa_unpack(wa_add2(ls2[2], ls2[3]), b0, b1);
       l += (a0 + a1) + (b0 + b1);
     }
-    if (ok) ok = mbar_wait(o_final(t), 0, abort_flag, p.status, ST_TIMEOUT_SOFTMAX);
-    if (ok) {
+    if (ok && hi > lo) ok = mbar_wait(o_final(t), 0, abort_flag, p.status, ST_TIMEOUT_SOFTMAX);
+    if (ok && hi > lo) {
       tc_fence_after();
       const float inv = l > 0.f ? 1.f / l : 0.f;
       const int qr = t * 128 + row;

@@ -36,7 +36,8 @@ TOL = {torch.float32: 3e-6, torch.bfloat16: 8e-3}
 
 # --------------------------------------------------------------------------- residual stream + norm
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
-@pytest.mark.parametrize("n,d,groups", [(3, 64, 1), (5, 96, 3), (2, 1000, 8), (700, 40, 5), (4, 4096, 2), (3, 90, 45), (2, 72, 36), (1, 16384, 4)])
+@pytest.mark.parametrize("n,d,groups", [(3, 64, 1), (5, 96, 3), (2, 1000, 8), (700, 40, 5), (4, 4096, 2), (3, 90, 45), (2, 72, 36), (1, 16384, 4),
+                                        (300, 512, 2), (310, 2056, 1), (297, 4096, 2), (300, 8192, 2), (299, 48, 2)])
 def test_residual_norm_sum_norm_and_embedding(dtype, n, d, groups):
     g = _gen(d)
     vocab = 50
@@ -60,22 +61,22 @@ def test_residual_norm_sum_norm_and_embedding(dtype, n, d, groups):
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
-@pytest.mark.parametrize("top", [1, 3])
-def test_residual_norm_dispatch_and_combine(dtype, top):
+@pytest.mark.parametrize("top,n,groups", [(1, 37, 4), (3, 37, 4), (3, 400, 2), (2, 400, 1)])
+def test_residual_norm_dispatch_and_combine(dtype, top, n, groups):
     g = _gen(top)
-    n, d = 37, 136
+    d = 136
     x0 = torch.randn(n, d, generator=g)
     gamma = torch.randn(d, generator=g).to(dtype)
     rows = torch.randperm(n * top, generator=g).to(torch.int32)
     x = x0.to(DEV)
     hs = torch.zeros(n * top, sops.pad8(d), dtype=dtype, device=DEV)
-    sops.residual_norm_(x, gamma.to(DEV), 4, 1e-6, hs, rows.to(DEV))
-    want = orc.grouped_rms_norm(x0.double(), gamma.double(), 1e-6, 4)
+    sops.residual_norm_(x, gamma.to(DEV), groups, 1e-6, hs, rows.to(DEV))
+    want = orc.grouped_rms_norm(x0.double(), gamma.double(), 1e-6, groups)
     _close(hs[:, :d][rows.long().to(DEV)].reshape(n, top, d), want[:, None].expand(n, top, d), TOL[dtype], "dispatch")
     y = torch.randn(n * top, d, generator=g)
     ys = torch.empty_like(y)
     ys[rows.long()] = y                                   # expert order
-    sops.residual_norm_(x, None, 4, 1e-6, y=ys.to(dtype).to(DEV), y_rows=rows.to(DEV), weight=1.0 / top)
+    sops.residual_norm_(x, None, groups, 1e-6, y=ys.to(dtype).to(DEV), y_rows=rows.to(DEV), weight=1.0 / top)
     _close(x, x0.double() + y.to(dtype).double().reshape(n, top, d).sum(1) / top, 2e-6, "combine")
 
 
