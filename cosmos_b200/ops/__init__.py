@@ -138,10 +138,12 @@ STATUS_MESSAGES = {
     4: "timeout: softmax waiting for scores",
     5: "timeout: waiting for a peer signal",
     6: "bad argument",
-    7: "index out of range (bounds-checked build)",
+    7: "index out of range",
 }
 STATUS_SITES = {1: "kv_cache_write slot", 2: "decode_qkv_post slot", 3: "paged_decode page id",
-                4: "paged_decode (tensor-core) page id", 15: "self-test"}
+                4: "paged_decode (tensor-core) page id", 5: "decoder stack token id", 6: "decoder stack cache slot",
+                7: "windowed attention page id", 8: "expert id of a routing table", 9: "expert-sorted row",
+                15: "self-test"}
 
 
 def check_status(reset: bool = True) -> None:

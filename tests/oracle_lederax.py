@@ -9,7 +9,7 @@ import torch
 
 
 def grouped_rms_norm(x, w, eps, groups):
-    """Each of `groups` equal consecutive parts of the last axis is divided by its own root mean square."""
+    """RMS norm over blocks of the last axis: x viewed as [.., groups, d / groups], normed along the last of these, times w."""
     parts = x.reshape(*x.shape[:-1], groups, x.shape[-1] // groups)
     parts = parts / torch.sqrt((parts * parts).mean(-1, keepdim=True) + eps)
     return parts.reshape(x.shape) * w

@@ -28,7 +28,7 @@ CONFIGS = {
     # one expert that everybody uses; all experts used by everybody
     "all_experts": config([layer(experts=1, top=1, ff=8), layer(experts=4, top=4, ff=16)], width=32, groups=8, scale=1.0),
     # shapes that the tensor-core kernels take (with bf16 on a GPU)
-    "tc": config([layer(heads=8, kv=2, dim=64, vdim=64, window=40), layer(heads=4, kv=2, dim=40, vdim=64, window=96, experts=7, top=2, ff=72),
+    "tc": config([layer(heads=4, kv=2, dim=64, vdim=64, window=40), layer(heads=16, kv=2, dim=40, vdim=64, window=90, experts=7, top=2, ff=72),
                   layer(heads=2, kv=2, dim=128, vdim=64, window=33)], vocab=200, width=192, groups=2),
 }
 

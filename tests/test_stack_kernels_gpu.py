@@ -231,7 +231,7 @@ PORTIONS = [
     (torch.float32, 3, 1, 50, 33, 5, 64, (70, 40)),
     (torch.float32, 2, 2, 130, 200, 16, 1, (19,)),
     (torch.bfloat16, 4, 2, 20, 36, 8, 9, (40, 3)),
-    (torch.bfloat16, 4, 2, 64, 64, 32, 96, (300, 129, 2)),
+    (torch.bfloat16, 4, 2, 64, 56, 32, 90, (300, 129, 2)),
     (torch.bfloat16, 2, 1, 128, 128, 16, 128, (400,)),
     (torch.bfloat16, 3, 3, 72, 40, 8, 33, (150, 77)),
     (torch.bfloat16, 2, 2, 40, 128, 64, 257, (600,)),
@@ -265,7 +265,7 @@ DECODE = [
     (torch.float32, 4, 2, 24, 40, 4, 7, (30, 1, 17)),
     (torch.float32, 5, 1, 50, 33, 5, 64, (70, 40)),
     (torch.bfloat16, 6, 2, 64, 64, 32, 40, (90, 41, 40, 39)),      # group of 3: CUDA-core kernel
-    (torch.bfloat16, 8, 2, 64, 64, 32, 96, (300, 97, 96, 95, 1)),
+    (torch.bfloat16, 8, 4, 64, 48, 32, 90, (300, 91, 90, 89, 1)),
     (torch.bfloat16, 8, 1, 128, 128, 16, 128, (400, 129, 5)),
     (torch.bfloat16, 4, 2, 72, 40, 8, 33, (150, 34, 33)),
     (torch.bfloat16, 2, 2, 40, 128, 64, 257, (600, 258, 257)),
