@@ -7,7 +7,7 @@ sizes README.md:79-85: Nano 16B = 2 x 8B towers, Super 64B = 2 x 32B towers).
 from __future__ import annotations
 
 from dataclasses import asdict, dataclass, field, replace
-from typing import Dict, List, Optional, Tuple
+from typing import Dict, List, Optional, Tuple, Union
 
 
 @dataclass
@@ -108,8 +108,10 @@ def super_config(**kw) -> MoTConfig:
 @dataclass(frozen=True)
 class AttentionSpec:
     """Attention mixer of a stack layer. The optional mechanisms are switches, so that another design can combine them
-    differently: sliding window (None = unlimited), distance bias `r1 ln(1 + r2 (i - j))` per head, RMS norm of each
-    value head, mixing of the values with those of an earlier layer, q/k/v biases."""
+    differently: sliding window (None = unlimited), distance bias `r1 ln(1 + r2 (i - j))` per head with learned r1, r2 or the
+    fixed linear bias `2^(-8 (h + 1) / heads) (i - j)`, RMS norm of each value head, mixing of the values with those of an
+    earlier layer, q/k/v biases, RMS norm over the whole query / key projection, keys that serve as values, a temperature
+    on the queries that grows with the logarithm of the position."""
     heads: int
     kv_heads: int
     dim: int                      # query / key head size
@@ -117,13 +119,67 @@ class AttentionSpec:
     scale: float
     window: Optional[int] = None  # keys seen by a query, itself included
     distance_bias: bool = False
+    linear_bias: bool = False
     value_norm: bool = False
     value_mix: bool = False       # the first such layer gives its values, the others mix them in
     qkv_bias: bool = False
+    qk_norm: bool = False         # over all heads at once
+    key_values: bool = False      # v = the projected keys before their norm
+    q_temp: Optional[Tuple[float, int]] = None   # (coef, every): q *= 1 + coef ln(floor((p + 1) / every) + 1)
 
     @property
     def qkv_cols(self) -> int:
-        return self.heads * self.dim + self.kv_heads * (self.dim + self.vdim)
+        return self.heads * self.dim + self.kv_heads * (self.dim + (0 if self.key_values else self.vdim))
+
+    def check(self) -> None:
+        if min(self.heads, self.kv_heads, self.dim, self.vdim) < 1 or self.heads % self.kv_heads:
+            raise ValueError("heads must be a positive multiple of kv_heads")
+        if self.window is not None and self.window < 1:
+            raise ValueError("the window holds at least the token itself")
+        if self.key_values and self.dim != self.vdim:
+            raise ValueError("keys serve as values: dim and vdim must be equal")
+        if self.q_temp is not None and self.q_temp[1] < 1:
+            raise ValueError("the query temperature needs a positive step")
+
+
+@dataclass(frozen=True)
+class MatrixMemorySpec:
+    """mLSTM mixer: a [dim, vdim] matrix memory per head with exponential input gate and sigmoid forget gate, both gates'
+    pre-activations soft-capped at `gate_cap`; heads normed, weighted and gated at the output."""
+    heads: int
+    dim: int
+    vdim: int
+    gate_cap: float
+
+    def check(self) -> None:
+        if min(self.heads, self.dim, self.vdim) < 1 or not self.gate_cap > 0:
+            raise ValueError("a matrix memory needs positive sizes and a positive gate cap")
+
+
+@dataclass(frozen=True)
+class SelectiveScanSpec:
+    """Mamba mixer: `inner` channels with `state` states each, a causal convolution of `conv` taps ahead of the scan, step
+    sizes from a projection of rank `dt_rank`."""
+    inner: int
+    state: int
+    dt_rank: int
+    conv: int
+
+    def check(self) -> None:
+        if min(self.inner, self.state, self.dt_rank, self.conv) < 1:
+            raise ValueError("a selective scan needs positive sizes")
+
+
+@dataclass(frozen=True)
+class ParallelSpec:
+    """Attention and a matrix memory side by side on the same input: half the sum of the two outputs, each RMS-normed over the
+    model width with a weight of its own."""
+    left: AttentionSpec
+    right: MatrixMemorySpec
+
+    def check(self) -> None:
+        self.left.check()
+        self.right.check()
 
 
 @dataclass(frozen=True)
@@ -134,16 +190,38 @@ class MoESpec:
     top: int
     ff: int
 
+    def check(self) -> None:
+        if not 1 <= self.top <= self.experts:
+            raise ValueError("top must be between 1 and the number of experts")
+
+
+@dataclass(frozen=True)
+class DenseSpec:
+    """down(silu(gate(h)) * up(h)) without biases."""
+    ff: int
+
+    def check(self) -> None:
+        if self.ff < 1:
+            raise ValueError("the feed-forward needs a positive size")
+
 
 @dataclass(frozen=True)
 class StackLayerSpec:
-    mixer: AttentionSpec
-    mlp: Optional[MoESpec] = None
+    mixer: Union[AttentionSpec, ParallelSpec, SelectiveScanSpec]
+    mlp: Union[MoESpec, DenseSpec, None] = None
+    weights_of: Optional[int] = None   # uses another layer's weights (with a cache and state of its own)
+
+    @property
+    def attention(self) -> Optional[AttentionSpec]:
+        """The attention of this layer, if it has one."""
+        return self.mixer.left if isinstance(self.mixer, ParallelSpec) else self.mixer if isinstance(self.mixer, AttentionSpec) else None
 
 
 @dataclass
 class StackConfig:
-    """A decoder whose layers are listed one by one (models/stack.py)."""
+    """A decoder whose layers are listed one by one (models/stack.py). `order`: "serial" = x += mixer(norm1 x), then
+    x += mlp(norm2 x); "parallel" = x += mixer(norm1 x) + mlp(norm2 x), both of the same x. `norm_add` is added to the stored
+    norm weights (1 for weights stored around zero)."""
     name: str
     architecture: str
     vocab_size: int
@@ -153,6 +231,10 @@ class StackConfig:
     norm_eps: float = 1e-6
     norm_groups: int = 1
     init_std: float = 0.02
+    order: str = "serial"
+    norm_add: float = 0.0
+    sinusoid: bool = False        # add the sinusoid of the position to the embedding
+    tied_head: bool = False
 
     @property
     def n_layers(self) -> int:
@@ -162,23 +244,43 @@ class StackConfig:
     def rms_eps(self) -> float:
         return self.norm_eps
 
+    def source_layer(self, i: int) -> int:
+        """The layer whose weights layer i uses."""
+        while self.layers[i].weights_of is not None:
+            i = self.layers[i].weights_of
+        return i
+
     def validate(self) -> "StackConfig":
         if self.vocab_size < 1 or self.d_model < 1 or self.norm_groups < 1 or self.d_model % self.norm_groups:
             raise ValueError("vocab and width must be positive and the width a multiple of the norm groups")
         first = None
         for i, layer in enumerate(self.layers):
-            m = layer.mixer
-            if min(m.heads, m.kv_heads, m.dim, m.vdim) < 1 or m.heads % m.kv_heads:
-                raise ValueError(f"layer {i}: heads must be a positive multiple of kv_heads")
-            if m.window is not None and m.window < 1:
-                raise ValueError(f"layer {i}: the window holds at least the token itself")
-            if m.value_mix:
+            m, j = layer.mixer, layer.weights_of
+            try:
+                m.check()
+                if layer.mlp is not None:
+                    layer.mlp.check()
+            except ValueError as e:
+                raise ValueError(f"layer {i}: {e}") from None
+            if j is not None:
+                if not 0 <= j < self.n_layers or j == i:
+                    raise ValueError(f"layer {i}: there is no layer {j} whose weights it could use")
+                seen = {i}
+                while j is not None and j not in seen:
+                    seen.add(j)
+                    j = self.layers[j].weights_of
+                src = self.layers[layer.weights_of]
+                if j is not None or (src.mixer, src.mlp) != (m, layer.mlp):
+                    raise ValueError(f"layer {i}: shared weights need an equal layer that leads to weights of its own")
+            if isinstance(m, AttentionSpec) and m.value_mix:
                 if first is None:
                     first = m
                 elif (m.kv_heads, m.vdim) != (first.kv_heads, first.vdim):
                     raise ValueError(f"layer {i}: mixed values need the first mixing layer's kv_heads and vdim")
-            if layer.mlp is not None and not 1 <= layer.mlp.top <= layer.mlp.experts:
-                raise ValueError(f"layer {i}: top must be between 1 and the number of experts")
+            if self.order == "serial" and not (isinstance(m, AttentionSpec) and isinstance(layer.mlp, (MoESpec, type(None)))):
+                raise ValueError(f"layer {i}: serial layers take attention and table-routed experts")
+            if self.order == "parallel" and (isinstance(m, AttentionSpec) or isinstance(layer.mlp, MoESpec)):
+                raise ValueError(f"layer {i}: parallel layers take a scan or attention beside a matrix memory, and a dense feed-forward")
         return self
 
     def to_dict(self) -> Dict:
@@ -220,8 +322,56 @@ def lederax_config_to_dict(cfg: StackConfig) -> Dict:
             "embedding": {"scale": cfg.embed_scale}, "norm": {"eps": cfg.norm_eps, "groups": cfg.norm_groups}, "layers": layers}
 
 
+def mererax_config_from_dict(doc: Dict, name: str = "Mererax") -> StackConfig:
+    """config.json of a Mererax model."""
+    layers = []
+    for i, entry in enumerate(doc["layers"]):
+        m, f = entry["mixer"], entry.get("mlp")
+        if entry["type"] == "parallel":
+            a, r = m["left"], m["right"]
+            temp = a.get("q_temp")
+            left = AttentionSpec(heads=int(a["heads"]), kv_heads=int(a["kv_heads"]), dim=int(a["dim"]), vdim=int(a.get("vdim", a["dim"])),
+                                 scale=float(a["scale"]), linear_bias=True, qk_norm=True, key_values=True,
+                                 q_temp=(float(temp["coef"]), int(temp["every"])) if temp else None)
+            mixer = ParallelSpec(left, MatrixMemorySpec(heads=int(r["heads"]), dim=int(r["dim"]), vdim=int(r["vdim"]),
+                                                        gate_cap=float(r["gate_cap"])))
+        elif entry["type"] == "mamba1":
+            mixer = SelectiveScanSpec(inner=int(m["inner"]), state=int(m["state"]), dt_rank=int(m["dt_rank"]), conv=int(m["conv"]))
+        else:
+            raise ValueError(f"layer {i}: unknown mixer type {entry['type']!r}")
+        if f is not None and f.get("kind") != "dense":
+            raise ValueError(f"layer {i}: unknown feed-forward kind {f.get('kind')!r}")
+        of = entry.get("weights_of")
+        layers.append(StackLayerSpec(mixer, None if f is None else DenseSpec(int(f["ff"])), None if of is None else int(of)))
+    return StackConfig(name=name, architecture="Mererax", vocab_size=int(doc["vocab"]), d_model=int(doc["width"]), layers=tuple(layers),
+                       embed_scale=float(doc["embedding"]["scale"]), norm_eps=float(doc["norm"]["eps"]), order="parallel", norm_add=1.0,
+                       sinusoid=True, tied_head=True).validate()
+
+
+def mererax_config_to_dict(cfg: StackConfig) -> Dict:
+    layers = []
+    for layer in cfg.layers:
+        m, f = layer.mixer, layer.mlp
+        if isinstance(m, ParallelSpec):
+            a, r = m.left, m.right
+            left = {"heads": a.heads, "kv_heads": a.kv_heads, "dim": a.dim, "vdim": a.vdim, "scale": a.scale}
+            if a.q_temp is not None:
+                left["q_temp"] = {"coef": a.q_temp[0], "every": a.q_temp[1]}
+            entry = {"type": "parallel", "mixer": {"left": left, "right": {"heads": r.heads, "dim": r.dim, "vdim": r.vdim,
+                                                                           "gate_cap": r.gate_cap}}}
+        else:
+            entry = {"type": "mamba1", "mixer": {"inner": m.inner, "state": m.state, "dt_rank": m.dt_rank, "conv": m.conv}}
+        entry["mlp"] = None if f is None else {"kind": "dense", "ff": f.ff}
+        if layer.weights_of is not None:
+            entry["weights_of"] = layer.weights_of
+        layers.append(entry)
+    return {"architecture": "Mererax", "vocab": cfg.vocab_size, "width": cfg.d_model, "embedding": {"scale": cfg.embed_scale},
+            "norm": {"eps": cfg.norm_eps}, "layers": layers}
+
+
 # architecture name in config.json -> (reader, writer)
-ARCHITECTURES = {"Lederax": (lederax_config_from_dict, lederax_config_to_dict)}
+ARCHITECTURES = {"Lederax": (lederax_config_from_dict, lederax_config_to_dict),
+                 "Mererax": (mererax_config_from_dict, mererax_config_to_dict)}
 
 
 def stack_config_from_dir(path) -> Optional[StackConfig]:
@@ -259,9 +409,37 @@ def lederax_8b_config(n_layers: int = 36, **kw) -> StackConfig:
                                   experts=32, top=4, ff=4608, vocab_size=151936), **kw)
 
 
+def mererax_preset(name: str, d_model: int, n_layers: int, heads: int, kv_heads: int, dim: int, mem_heads: int, mem_dim: int,
+                   mem_vdim: int, inner: int, state: int, dt_rank: int, ff: int, vocab_size: int, every: int = 1024,
+                   period: int = 3) -> StackConfig:
+    """Scan layers with an attention / memory layer as the last of every `period`."""
+    par = StackLayerSpec(ParallelSpec(AttentionSpec(heads=heads, kv_heads=kv_heads, dim=dim, vdim=dim, scale=dim ** -0.5, linear_bias=True,
+                                                    qk_norm=True, key_values=True, q_temp=(0.1, every)),
+                                      MatrixMemorySpec(heads=mem_heads, dim=mem_dim, vdim=mem_vdim, gate_cap=15.0)), DenseSpec(ff))
+    scan = StackLayerSpec(SelectiveScanSpec(inner=inner, state=state, dt_rank=dt_rank, conv=4), DenseSpec(ff))
+    return StackConfig(name=name, architecture="Mererax", vocab_size=vocab_size, d_model=d_model,
+                       layers=tuple(par if i % period == period - 1 else scan for i in range(n_layers)), embed_scale=d_model ** 0.5,
+                       order="parallel", norm_add=1.0, sinusoid=True, tied_head=True).validate()
+
+
+def mererax_tiny_config(n_layers: int = 3, **kw) -> StackConfig:
+    """Toy model of the CPU tests and examples (byte-level tokenizer)."""
+    return replace(mererax_preset("mererax-tiny", d_model=80, n_layers=n_layers, heads=4, kv_heads=2, dim=20, mem_heads=3, mem_dim=12,
+                                  mem_vdim=28, inner=112, state=10, dt_rank=6, ff=136, vocab_size=300, every=16), **kw)
+
+
+def mererax_8b_config(n_layers: int = 36, **kw) -> StackConfig:
+    """Layers as wide as Cosmos3-Nano's Reasoner tower: attention 32 / 8 heads of 128 beside 8 memories of 256 x 512, scans of
+    8192 channels x 16 states, SwiGLU of 12288."""
+    return replace(mererax_preset("mererax-8b", d_model=4096, n_layers=n_layers, heads=32, kv_heads=8, dim=128, mem_heads=8, mem_dim=256,
+                                  mem_vdim=512, inner=8192, state=16, dt_rank=256, ff=12288, vocab_size=151936), **kw)
+
+
 MODEL_REGISTRY = {
     "lederax-tiny": lederax_tiny_config,
     "lederax-8b": lederax_8b_config,
+    "mererax-tiny": mererax_tiny_config,
+    "mererax-8b": mererax_8b_config,
     "tiny": tiny_config,
     "tiny128": tiny128_config,
     "Cosmos3-Nano": nano_config,

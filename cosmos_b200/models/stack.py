@@ -7,7 +7,7 @@ prompts of several sequences, or one new token of every decode slot) against the
 trace runner all go through it. Launches per layer on CUDA bf16:
   q/k/v GEMM (+ bias) -> value norm + mixing + cache write -> paged windowed attention -> out-projection GEMM
   -> residual add + norm + dispatch into expert order -> up GEMM (+ gelu) -> down GEMM -> combine + residual add + norm
-For a few rows (decode) the GEMMs split K and leave fp32 partial sums that the kernel behind each of them reduces. The
+(layers in serial order; those in parallel order, with recurrent mixers, are in stack_parallel.py). For a few rows (decode) the GEMMs split K and leave fp32 partial sums that the kernel behind each of them reduces. The
 experts depend on the token ids alone, so one launch at the start of the step routes every layer.
 """
 from __future__ import annotations
@@ -20,25 +20,26 @@ import torch
 import torch.nn as nn
 
 from .. import ops
-from ..config import MODEL_REGISTRY, StackConfig, StackLayerSpec, get_model_config, stack_config_from_dir
+from ..config import MODEL_REGISTRY, AttentionSpec, StackConfig, StackLayerSpec, get_model_config, stack_config_from_dir
 from ..ops import stack as sops
-from ..ops.stack import pad8
+from ..ops.stack import StepRows, pad8
+from .stack_parallel import ParallelLayer, split_k
+from .stack_parallel import param as _param
 
 
 @dataclass
 class StepBatch:
     """The tokens of one step, in row order, and where they go. Portions: `tiles` [t, 4] int32 lists the query tiles.
-    Decode: `lens` [n] int32 holds every slot's length including its new token (0 = idle slot)."""
+    Decode: `lens` [n] int32 holds every slot's length including its new token (0 = idle slot). `rows`: the same for
+    recurrent layers."""
     tokens: torch.Tensor                 # [n] int64
     slots: torch.Tensor                  # [n] int64 cache slots (page * page_size + offset)
     table: torch.Tensor                  # [sequences, max_pages] int32
     tiles: Optional[Dict[int, torch.Tensor]] = None   # query tiles by rows per tile
     lens: Optional[torch.Tensor] = None
     max_len: Optional[int] = None        # host-known bound of `lens`
-
-
-def _param(shape, dtype, device) -> nn.Parameter:
-    return nn.Parameter(torch.zeros(shape, dtype=dtype, device=device), requires_grad=False)
+    positions: Optional[torch.Tensor] = None          # [n] int64
+    rows: Optional[StepRows] = None
 
 
 class StackLayer(nn.Module):
@@ -98,38 +99,60 @@ class StackModel(nn.Module):
     def __init__(self, cfg: StackConfig, dtype=torch.bfloat16, device="cpu"):
         super().__init__()
         self.cfg, self.dtype = cfg, dtype
-        d8 = pad8(cfg.d_model)
-        self.embed = _param((cfg.vocab_size, cfg.d_model), dtype, device)
-        self.layers = nn.ModuleList([StackLayer(cfg, s, dtype, device) for s in cfg.layers])
-        self.final_norm = _param((cfg.d_model,), dtype, device)
-        self.w_head = _param((pad8(cfg.vocab_size), d8), dtype, device)
-        self._moe = [i for i, s in enumerate(cfg.layers) if s.mlp is not None]
+        d8, v8 = pad8(cfg.d_model), pad8(cfg.vocab_size)
+        self.parallel = cfg.order == "parallel"
+        # a tied head is the embedding table itself, stored with the padding that the head's product needs
+        self.w_head = _param((v8, d8), dtype, device)
+        self.embed = self.w_head[:cfg.vocab_size, :cfg.d_model] if cfg.tied_head else _param((cfg.vocab_size, cfg.d_model), dtype, device)
+        kind = ParallelLayer if self.parallel else StackLayer
+        own = {i: kind(cfg, s, dtype, device) for i, s in enumerate(cfg.layers) if s.weights_of is None}
+        self.layers = nn.ModuleList([own[cfg.source_layer(i)] for i in range(cfg.n_layers)])
+        self.final_norm = _param((cfg.d_model,), torch.float32 if self.parallel else dtype, device)
+        self._moe = [] if self.parallel else [i for i, s in enumerate(cfg.layers) if s.mlp is not None]
         self._desc: Dict[Tuple, torch.Tensor] = {}
-        mixing = [i for i, s in enumerate(cfg.layers) if s.mixer.value_mix]
+        mixing = [i for i, s in enumerate(cfg.layers) if isinstance(s.mixer, AttentionSpec) and s.mixer.value_mix]
         self.first_mix = mixing[0] if mixing else -1
+        self.pos_turns = sops.sinusoid_turns(cfg.d_model, device) if cfg.sinusoid else None
 
     @property
     def device(self) -> torch.device:
-        return self.embed.device
+        return self.w_head.device
 
     # ------------------------------------------------------------------ weights
-    def checkpoint_views(self) -> Dict[str, torch.Tensor]:
-        out = {"embed": self.embed, "final.norm": self.final_norm,
-               "head": self.w_head[:self.cfg.vocab_size, :self.cfg.d_model]}
+    def checkpoint_views(self) -> Dict[str, object]:
+        """Checkpoint tensor name -> the storage that holds it (a tuple: parts stacked along the rows)."""
+        out: Dict[str, object] = {"embed": self.embed, "final.norm": self.final_norm}
+        if not self.cfg.tied_head:
+            out["head"] = self.w_head[:self.cfg.vocab_size, :self.cfg.d_model]
         for i, layer in enumerate(self.layers):
-            out.update(layer.checkpoint_views(f"l{i}."))
+            if self.cfg.layers[i].weights_of is None:
+                out.update(layer.checkpoint_views(f"l{i}."))
         return out
+
+    def finish(self) -> "StackModel":
+        """Values derived from the weights (after loading or drawing them)."""
+        if self.parallel:
+            for layer in self.layers:
+                layer.finish()
+        return self
 
     @torch.no_grad()
     def load(self, model_dir) -> "StackModel":
         from ..ckpt import safetensors_io as sio
 
-        targets = {k: v.data for k, v in self.checkpoint_views().items()}
+        views = self.checkpoint_views()
+        stacked = {k: v for k, v in views.items() if isinstance(v, tuple)}
+        targets = {k: v.data for k, v in views.items() if k not in stacked}
+        for k, parts in stacked.items():
+            targets[k] = torch.empty(sum(p.shape[0] for p in parts), *parts[0].shape[1:], dtype=parts[0].dtype, device=parts[0].device)
         unused = f"l{self.first_mix}.mix.vmix"   # the first mixing layer has nothing to mix with
         if unused in targets and unused not in sio.tensor_files(model_dir):
             del targets[unused]
         sio.load_into(model_dir, targets)
-        return self.check_tables()
+        for k, parts in stacked.items():
+            for p, src in zip(parts, targets[k].split([p.shape[0] for p in parts])):
+                p.copy_(src)
+        return self.check_tables().finish()
 
     def check_tables(self) -> "StackModel":
         for i in self._moe:
@@ -144,45 +167,64 @@ class StackModel(nn.Module):
 
         from ..ckpt import safetensors_io as sio
 
-        half = {k: v.detach().to(torch.bfloat16) if v.is_floating_point() else v for k, v in self.checkpoint_views().items()}
+        whole = {k: torch.cat(v) if isinstance(v, tuple) else v for k, v in self.checkpoint_views().items()}
+        half = {k: v.detach().to(torch.bfloat16) if v.is_floating_point() else v for k, v in whole.items()}
         sio.save_sharded(half, model_dir)
         (Path(model_dir) / "config.json").write_text(json.dumps(self.cfg.to_dict(), indent=1))
 
     @torch.no_grad()
     def init_weights(self, seed: int = 0) -> "StackModel":
-        """Random weights: N(0, init_std) matrices, unit norms, mild biases, random routing tables without repeats in a row."""
+        """Random weights: N(0, init_std) matrices, neutral norms, mild biases, random routing tables without repeats in a row,
+        decays and step sizes over the usual range of selective scans, forget gates mostly open."""
         dev, std = self.device, self.cfg.init_std
         g = torch.Generator(device=dev)
         g.manual_seed(seed)
-        for name, v in self.checkpoint_views().items():
+
+        def rand(v, lo, hi):
+            return torch.rand(v.shape, generator=g, device=dev) * (hi - lo) + lo
+
+        views = [(name, v) for name, vs in self.checkpoint_views().items() for v in (vs if isinstance(vs, tuple) else (vs,))]
+        for name, v in views:
             leaf = name.split(".")[-1]
-            if leaf in ("norm1", "norm2", "norm"):
+            if leaf in ("norm1", "norm2") or name == "final.norm":
+                v.fill_(1.0 - self.cfg.norm_add)
+            elif leaf in ("norm", "out") or leaf == "D":
                 v.fill_(1.0)
             elif leaf == "table":
                 e = self.cfg.layers[int(name[1:name.index(".")])].mlp.experts
                 v.copy_(torch.rand(v.shape[0], e, generator=g, device=dev).argsort(1)[:, :v.shape[1]].to(torch.int32))
             elif leaf in ("r1", "r2"):
-                v.copy_(torch.rand(v.shape, generator=g, device=dev) * 0.5 + 0.05)
+                v.copy_(rand(v, 0.05, 0.55))
             elif leaf == "vmix":
                 v.fill_(0.5)
+            elif leaf == "A_log":
+                v.copy_(torch.arange(1, v.shape[1] + 1, device=dev).float().log().expand_as(v))
+            elif name.endswith("mix.dt.b"):    # softplus of it between 0.001 and 0.1
+                v.copy_(torch.expm1(torch.exp(rand(v, -6.9, -2.3))).log())
+            elif name.endswith("right.f.b"):
+                v.copy_(rand(v, 3.0, 6.0))
+            elif leaf == "conv":
+                v.copy_(rand(v, -0.5, 0.5))
             else:
                 v.copy_(torch.randn(v.shape, generator=g, device=dev, dtype=torch.float32) * std)
-        return self
+        return self.finish()
 
     def kv_shapes(self) -> List[Tuple[int, int, int]]:
-        return [(s.mixer.kv_heads, s.mixer.dim, s.mixer.vdim) for s in self.cfg.layers]
+        """(kv heads, key size, value size) of every layer; no heads = a layer without attention."""
+        att = [s.attention for s in self.cfg.layers]
+        return [(0, 0, 0) if a is None else (a.kv_heads, a.dim, a.vdim) for a in att]
+
+    def state_shapes(self) -> List[Dict[str, Tuple]]:
+        """Per layer: name -> (shape, dtype) of what a sequence carries from token to token beside the paged cache."""
+        return [layer.mixer.state_shapes(self.dtype) for layer in self.layers] if self.parallel else []
 
     def tile_sizes(self, page_size: int) -> List[int]:
-        """Query rows per attention tile of every layer (which kernel takes its shape)."""
-        return [sops.attn_tile_rows(s.mixer.heads, s.mixer.kv_heads, s.mixer.dim, s.mixer.vdim, page_size, self.dtype,
-                                    self.device) for s in self.cfg.layers]
+        """Query rows per attention tile of every layer (which kernel takes its shape); 0 = no attention."""
+        att = [s.attention for s in self.cfg.layers]
+        return [0 if a is None else sops.attn_tile_rows(a.heads, a.kv_heads, a.dim, a.vdim, page_size, self.dtype, self.device)
+                for a in att]
 
     # ------------------------------------------------------------------ the step
-    def _split_k(self, n: int, w: torch.Tensor) -> bool:
-        """Whether a product of n rows is skinny enough that the GEMM splits K (and a consumer can reduce the sums)."""
-        return (w.is_cuda and w.dtype == torch.bfloat16 and ops.load_extension()
-                and torch.ops.cosmos_b200.gemm_pick_k_splits(n, w.shape[0], w.shape[1], ops.EPI_PLAIN) > 1)
-
     def _route(self, tokens: torch.Tensor) -> Optional[sops.Routing]:
         if not self._moe:
             return None
@@ -203,7 +245,7 @@ class StackModel(nn.Module):
         """Mixer of layer li on the normed rows h [n, d]: -> y [n, >= d] (or fp32 partial sums)."""
         layer, m, n = self.layers[li], self.cfg.layers[li].mixer, h.shape[0]
         w = layer.w_qkv[:, :layer.d]
-        if self._split_k(n, w):
+        if split_k(n, w):
             qkv = sops.gemm_partial(h, w)
         else:
             qkv = ops.gemm(h, w, layer.b_qkv)
@@ -218,7 +260,7 @@ class StackModel(nn.Module):
         o = sops.window_attn(q, cache.k[li], cache.v[li], batch.table, m.scale, m.window, layer.r1, layer.r2,
                              None if batch.tiles is None else batch.tiles[tile_rows], tile_rows, batch.lens, batch.max_len)
         w = layer.w_o[:, :layer.o_cols]
-        return sops.gemm_partial(o, w) if self._split_k(n, w) else ops.gemm(o, w)
+        return sops.gemm_partial(o, w) if split_k(n, w) else ops.gemm(o, w)
 
     def _experts(self, li: int, hs: torch.Tensor, rt: sops.Routing, k: int, n: int) -> torch.Tensor:
         """Feed-forward of layer li on the dispatched rows hs [n * top, d]: -> the experts' outputs in the same order."""
@@ -236,6 +278,8 @@ class StackModel(nn.Module):
                      layers_out: Optional[List[torch.Tensor]] = None) -> torch.Tensor:
         """Logits [len(rows), vocab] of the chosen rows (None = all). `layers_out` receives the residual stream after every
         layer (debugging)."""
+        if self.parallel:
+            return self._parallel_step(batch, cache, tile_sizes, rows, layers_out)
         cfg, dev, dt = self.cfg, self.device, self.dtype
         n, d, g, eps = batch.tokens.shape[0], cfg.d_model, cfg.norm_groups, cfg.norm_eps
         x = torch.empty(n, d, dtype=torch.float32, device=dev)
@@ -266,6 +310,39 @@ class StackModel(nn.Module):
             xr = x[rows]
             h = torch.empty(xr.shape[0], pad8(d), dtype=dt, device=dev)
             sops.residual_norm_(xr, self.final_norm, g, eps, h)
+        return ops.gemm(h[:, :d], self.w_head[:, :d])[:, :cfg.vocab_size]
+
+    def _parallel_step(self, batch: StepBatch, cache, tile_sizes: List[int], rows: Optional[torch.Tensor],
+                       layers_out: Optional[List[torch.Tensor]]) -> torch.Tensor:
+        cfg, dev, dt = self.cfg, self.device, self.dtype
+        n, d, eps, add = batch.tokens.shape[0], cfg.d_model, cfg.norm_eps, cfg.norm_add
+
+        def buffer(m: int = n) -> torch.Tensor:
+            return torch.empty(m, pad8(d), dtype=dt, device=dev)
+
+        x = torch.empty(n, d, dtype=torch.float32, device=dev)
+        first = dict(embed=self.embed, tokens=batch.tokens, embed_scale=cfg.embed_scale, pos_turns=self.pos_turns, positions=batch.positions)
+        branches, plain = [], None
+        for li, layer in enumerate(self.layers):
+            h1, h2 = buffer(), None if layer.norm2 is None else buffer()
+            sops.branch_norm_(x, eps, dt, branches, 0.5, plain, (layer.norm1, layer.norm2), add, (h1, h2), **first)
+            first = {}
+            if li > 0 and layers_out is not None:
+                layers_out.append(x.clone())
+            branches, plain = layer(h1[:, :d], None if h2 is None else h2[:, :d], batch, cache, li, tile_sizes[li])
+        h = None
+        if rows is None:
+            h = buffer()
+            sops.branch_norm_(x, eps, dt, branches, 0.5, plain, (self.final_norm,), add, (h,), **first)
+        else:           # only the asked rows need the final norm and the head
+            sops.branch_norm_(x, eps, dt, branches, 0.5, plain, **first)
+            if rows.shape[0] > 0:
+                h = buffer(rows.shape[0])
+                sops.branch_norm_(x[rows], eps, dt, gammas=(self.final_norm,), gamma_add=add, hs=(h,))
+        if layers_out is not None and cfg.n_layers > 0:
+            layers_out.append(x.clone())
+        if h is None:   # a portion in the middle of a prompt
+            return torch.empty(0, cfg.vocab_size, dtype=dt, device=dev)
         return ops.gemm(h[:, :d], self.w_head[:, :d])[:, :cfg.vocab_size]
 
 

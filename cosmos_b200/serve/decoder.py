@@ -31,7 +31,7 @@ from .. import ops
 from ..config import MoTConfig, get_model_config
 from ..models import rope
 from ..models.stack import StackModel, StepBatch
-from ..ops.stack import make_tiles
+from ..ops.stack import StepRows, make_conv_tiles, make_tiles
 from .paged import PagedKVCache
 
 
@@ -47,6 +47,7 @@ class StepDecoder:
         self.step_inc: Optional[torch.Tensor] = None  # int32 [B] of 0/1 set by the serving engine; None = all ones
         self.sampling: Optional[Dict[str, torch.Tensor]] = None  # see enable_sampling
         self.pos_delta: Optional[torch.Tensor] = None  # int64 [B]: rotary position minus cache position
+        self.state_slots: Optional[torch.Tensor] = None  # int32 [B]: recurrent-state slots (models that have such states)
 
     def _step_impl(self) -> None:
         raise NotImplementedError
@@ -119,6 +120,8 @@ class StepDecoder:
     def capture(self, warmup: int = 2) -> None:
         """Captures `_step_impl` into a CUDA graph. Warm-up steps run first (workspace and
         symmetric-memory set-up must not happen during capture); they advance the sequences."""
+        if self.cache.states is not None:
+            self.cache.states.frozen = True
         side = torch.cuda.Stream()
         side.wait_stream(torch.cuda.current_stream())
         with torch.cuda.stream(side):
@@ -388,7 +391,8 @@ class StackDecoder(StepDecoder):
         self.page_size = page_size
         pages_per_seq = (max_len + page_size - 1) // page_size
         self.cache = PagedKVCache(self.cfg.n_layers, 0, 0, num_pages or max_batch * pages_per_seq + 1, page_size,
-                                  pages_per_seq, model.dtype, self.device, kv_shapes=model.kv_shapes())
+                                  pages_per_seq, model.dtype, self.device, kv_shapes=model.kv_shapes(),
+                                  state_shapes=model.state_shapes(), state_slots=max_batch + 1)
         self.tile_sizes = model.tile_sizes(page_size)
         self._init_state()
 
@@ -400,7 +404,8 @@ class StackDecoder(StepDecoder):
             self.lens.add_(1)
         else:
             self.lens.add_(self.step_inc)
-        batch = StepBatch(self.tokens, slots, self.table, lens=self.lens, max_len=self.max_len)
+        rows = None if self.state_slots is None else StepRows(self.state_slots, lens=self.lens)
+        batch = StepBatch(self.tokens, slots, self.table, lens=self.lens, max_len=self.max_len, positions=pos, rows=rows)
         self._finish_step(self.model.forward_step(batch, self.cache, self.tile_sizes), self.tokens.shape[0])
 
     @torch.no_grad()
@@ -422,13 +427,23 @@ class StackDecoder(StepDecoder):
             raise ValueError("a portion reaches beyond the pages reserved for its sequence")
         row0 = [sum(counts[:i]) for i in range(len(counts))]
         rows = [row0[i] + w for i, e in enumerate(entries) for w in e[3]]
-        batch = StepBatch(toks.to(dev), slots.to(dev), table.to(dev))
+        batch = StepBatch(toks.to(dev), slots.to(dev), table.to(dev), positions=pos.to(dev))
+        state_slots = self.cache.state_slots(seqs)
+        if state_slots is not None:
+            batch.rows = StepRows(state_slots)
         if all(c == 1 for c in counts):   # one new token each: the decode kernels
             lens = torch.tensor([e[2] + 1 for e in entries], dtype=torch.int32)
             batch.lens, batch.max_len = lens.to(dev), int(lens.max())
+            if batch.rows is not None:
+                batch.rows.lens = batch.lens
         else:
+            def table_of(rows_) -> torch.Tensor:
+                return torch.tensor(rows_, dtype=torch.int32).to(dev)
+
             portions = [(i, row0[i], counts[i], entries[i][2]) for i in range(len(entries))]
-            batch.tiles = {r: torch.tensor(make_tiles(portions, r), dtype=torch.int32).to(dev) for r in set(self.tile_sizes)}
+            batch.tiles = {r: table_of(make_tiles(portions, r)) for r in set(self.tile_sizes) if r}
+            if batch.rows is not None:
+                batch.rows.portions, batch.rows.conv_tiles = table_of(portions), table_of(make_conv_tiles(portions))
         sel = torch.tensor(rows, dtype=torch.long).to(dev)
         return self.model.forward_step(batch, self.cache, self.tile_sizes, sel, layers_out)
 
@@ -445,6 +460,7 @@ class StackDecoder(StepDecoder):
                 lg = self.run_portions([(i, part, o, [len(part) - 1] if o + len(part) == len(ids) else [])])
             last.append(lg.float().argmax(-1))
         self.table, _ = self.cache.tables(self.seq_ids)
+        self.state_slots = self.cache.state_slots(self.seq_ids)
         self.lens = torch.tensor([len(p) for p in prompts], dtype=torch.int32, device=self.device)
         self.max_len = max(len(p) for p in prompts) + new_tokens
         self.tokens = torch.cat(last)

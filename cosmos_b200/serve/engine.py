@@ -96,6 +96,10 @@ class BatchEngine:
         self.dec.next_tokens = torch.zeros(max_batch, dtype=torch.long, device=dev)
         self.dec.step_inc = torch.zeros(max_batch, dtype=torch.int32, device=dev)
         self.dec.max_len = max_len
+        scratch = cache.state_slots([self.scratch_seq])   # idle slots leave states alone; they still need a valid number
+        self.scratch_state = 0 if scratch is None else int(scratch)
+        if scratch is not None:
+            self.dec.state_slots = torch.full((max_batch,), self.scratch_state, dtype=torch.int32, device=dev)
         self.dec.enable_sampling(max_batch)
         self.dec.pos_delta = torch.zeros(max_batch, dtype=torch.long, device=dev)
         self.noise_gen = torch.Generator(device=dev)
@@ -236,6 +240,8 @@ class BatchEngine:
         ids = ids.to(dev)
         real = torch.arange(max(lens), device=dev)[None] < len_t[:, None]
         dec.table[slot_idx] = table
+        if dec.state_slots is not None:
+            dec.state_slots[slot_idx] = dec.cache.state_slots([r.rid for r in group])
         # per-slot sampling state; the prompt tokens count as "seen" for the repetition penalty
         sp = dec.sampling
         for name, vals in (("temperature", [r.temperature for r in group]), ("top_p", [r.top_p for r in group]),
@@ -294,6 +300,8 @@ class BatchEngine:
         self.dec.lens[s] = 0
         self.dec.step_inc[s] = 0
         self.dec.tokens[s] = 0
+        if self.dec.state_slots is not None:
+            self.dec.state_slots[s] = self.scratch_state
         self.slots[s] = None
         self.finished[r.rid] = r
         if r.future is not None and not r.future.done():

@@ -5,12 +5,13 @@ Layout per layer: k_cache, v_cache [num_pages, Hkv_local, page_size, head_dim] b
 (page, head) are contiguous, which is what the decode kernel streams). A sequence
 owns a list of pages; token i of the sequence lives in page table[i // page_size] at offset
 i % page_size. Layers may differ in heads and head sizes, keys and values too (`kv_shapes`); the page tables are shared
-by all layers. Pages for the whole generation (prompt + max new tokens) can be reserved up front,
+by all layers. Recurrent layers keep fixed-size states instead (`StateCache`): a sequence owns one slot of every layer's
+state tensors from its first reservation to its release. Pages for the whole generation (prompt + max new tokens) can be reserved up front,
 which keeps the block table static during decode (a requirement for CUDA-graph replay).
 """
 from __future__ import annotations
 
-from typing import Optional, Sequence, Tuple
+from typing import Dict, List, Optional, Sequence, Tuple
 
 import torch
 
@@ -68,24 +69,81 @@ def make_allocator(num_blocks: int, block_size: int, max_blocks_per_seq: int):
     return _PyAllocator(num_blocks, block_size, max_blocks_per_seq)
 
 
+class StateCache:
+    """Recurrent states: per layer a dictionary of tensors [slots, ...], and one slot per live sequence. A slot is not cleared
+    when it changes hands: the layers take the state of a sequence at position 0 as zero."""
+
+    def __init__(self, shapes: Sequence[Dict[str, Tuple]], slots: int, device):
+        self.slots = slots
+        self.tensors = [{k: torch.zeros((slots, *shape), dtype=dtype, device=device) for k, (shape, dtype) in s.items()} for s in shapes]
+        self.free = list(range(slots - 1, -1, -1))
+        self.slot_of: Dict[int, int] = {}
+        self.frozen = False     # a captured graph holds the tensors' addresses
+
+    def acquire(self, seq_id: int) -> bool:
+        """Gives the sequence a slot (more slots are made while nothing holds the addresses). True = it has one now."""
+        if seq_id in self.slot_of:
+            return True
+        if not self.free:
+            if self.frozen:
+                return False
+            self._grow(2 * self.slots)
+        self.slot_of[seq_id] = self.free.pop()
+        return True
+
+    def _grow(self, slots: int) -> None:
+        for layer in self.tensors:
+            for k, t in layer.items():
+                layer[k] = torch.cat([t, t.new_zeros(slots - self.slots, *t.shape[1:])])
+        self.free = list(range(slots - 1, self.slots - 1, -1)) + self.free
+        self.slots = slots
+
+    def release(self, seq_id: int) -> None:
+        if seq_id in self.slot_of:
+            self.free.append(self.slot_of.pop(seq_id))
+
+
 class PagedKVCache:
     def __init__(self, n_layers: int, n_kv_heads: int, head_dim: int, num_pages: int, page_size: int,
                  max_pages_per_seq: int, dtype=torch.bfloat16, device="cuda",
-                 kv_shapes: Optional[Sequence[Tuple[int, int, int]]] = None):
-        """`kv_shapes`: (kv heads, key size, value size) of every layer; None = n_kv_heads x head_dim throughout."""
+                 kv_shapes: Optional[Sequence[Tuple[int, int, int]]] = None, state_shapes: Sequence[Dict[str, Tuple]] = (),
+                 state_slots: int = 0):
+        """`kv_shapes`: (kv heads, key size, value size) of every layer; None = n_kv_heads x head_dim throughout.
+        `state_shapes`: name -> (shape, dtype) of every layer's recurrent state, for models that have one."""
         self.n_layers, self.page_size, self.max_pages = n_layers, page_size, max_pages_per_seq
         self.alloc = make_allocator(num_pages, page_size, max_pages_per_seq)
         shapes = list(kv_shapes) if kv_shapes is not None else [(n_kv_heads, head_dim, head_dim)] * n_layers
         self.k = [torch.zeros((num_pages, h, page_size, kd), dtype=dtype, device=device) for h, kd, _ in shapes]
         self.v = [torch.zeros((num_pages, h, page_size, vd), dtype=dtype, device=device) for h, _, vd in shapes]
         self.device = torch.device(device)
+        self.states = StateCache(state_shapes, max(1, state_slots), device) if state_shapes else None
+
+    @property
+    def state(self) -> List[Dict[str, torch.Tensor]]:
+        return self.states.tensors if self.states is not None else []
 
     def reserve(self, seq_id: int, tokens: int) -> bool:
-        """Reserves pages for `tokens` more tokens of a sequence (False = pool exhausted)."""
-        return bool(self.alloc.extend(seq_id, tokens))
+        """Reserves pages for `tokens` more tokens of a sequence, and its state slot (False = pool exhausted)."""
+        if self.states is None:
+            return bool(self.alloc.extend(seq_id, tokens))
+        had = seq_id in self.states.slot_of
+        if not self.states.acquire(seq_id):
+            return False
+        ok = bool(self.alloc.extend(seq_id, tokens))
+        if not ok and not had:
+            self.states.release(seq_id)
+        return ok
 
     def release(self, seq_id: int) -> None:
         self.alloc.release(seq_id)
+        if self.states is not None:
+            self.states.release(seq_id)
+
+    def state_slots(self, seq_ids: Sequence[int]) -> Optional[torch.Tensor]:
+        """int32 [n] on the device: the state slots of sequences (None for models without states)."""
+        if self.states is None:
+            return None
+        return torch.tensor([self.states.slot_of[s] for s in seq_ids], dtype=torch.int32).to(self.device)
 
     def tables(self, seq_ids: Sequence[int]):
         """(block_table [n, max_pages] int32, reserved lengths [n] int32) on the cache's device."""

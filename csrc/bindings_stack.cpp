@@ -164,11 +164,14 @@ Tensor window_attn(const Tensor& q, const Tensor& k_cache, const Tensor& v_cache
   a.table = table.data_ptr<int>(); a.max_pages = (int)table.size(1); a.n_seqs = (int)table.size(0);
   a.scale = (float)scale; a.window = (int)window;
   TORCH_CHECK(window >= 1, "window must be at least 1");
-  if (has(r1)) {
-    TORCH_CHECK(has(r2) && r1->is_cuda() && r2->is_cuda() && r1->scalar_type() == at::kFloat && r2->scalar_type() == at::kFloat &&
-                    r1->is_contiguous() && r2->is_contiguous() && r1->numel() == a.H && r2->numel() == a.H, "r1, r2 must be fp32 [H]");
-    a.r1 = r1->data_ptr<float>(); a.r2 = r2->data_ptr<float>();
-  }
+  auto per_head = [&](const OptT& t, const char* name) -> const float* {
+    if (!has(t)) return nullptr;
+    TORCH_CHECK(t->is_cuda() && t->scalar_type() == at::kFloat && t->is_contiguous() && t->numel() == a.H, name, " must be fp32 [H]");
+    return t->data_ptr<float>();
+  };
+  a.r1 = per_head(r1, "r1");
+  a.r2 = per_head(r2, "r2");   // none: a linear bias
+  TORCH_CHECK(a.r1 || !a.r2, "r2 without r1");
   // a row is padded to a multiple of 8 elements: the output projection reads it with 16-byte rows
   const int64_t cols = (int64_t)a.H * a.vdim, ld = (cols + 7) / 8 * 8;
   Tensor out = at::empty({q.size(0), ld}, q.options());
@@ -292,6 +295,215 @@ Tensor gemm_partial(const Tensor& a_, const Tensor& w) {
   return part;
 }
 
+// ---------------------------------------------------------------- parallel layers and recurrent mixers
+// Rows for a kernel of element type `f32 ? float : bf16`: finished values [n, >= cols] of that type, or fp32 values
+// [n, >= cols] / split-K partial sums [splits, n, >= cols].
+cosmos::RowSource row_source(const Tensor& t, bool f32, int64_t n, int64_t cols, const char* name) {
+  TORCH_CHECK(t.is_cuda() && (t.dim() == 2 || t.dim() == 3) && t.stride(-1) == 1 && t.size(-2) >= n && t.size(-1) >= cols, name,
+              " must be [n, cols] rows or [splits, n, cols] partial sums");
+  cosmos::RowSource s;
+  s.p = t.data_ptr(); s.ld = t.stride(-2);
+  if (t.dim() == 2 && is_f32(t, name) == f32) return s;
+  TORCH_CHECK(t.scalar_type() == at::kFloat, name, ": partial sums must be fp32");
+  s.k_splits = t.dim() == 3 ? (int)t.size(0) : 1;
+  s.split_stride = t.dim() == 3 ? t.stride(0) : 0;
+  return s;
+}
+const float* f32_vec(const Tensor& t, int64_t n, const char* name) {
+  TORCH_CHECK(t.is_cuda() && t.scalar_type() == at::kFloat && t.is_contiguous() && t.numel() == n, name, " must be contiguous fp32 with ",
+              n, " entries");
+  return t.data_ptr<float>();
+}
+// portions int32 [p, 4], or lens int32 [n] of a decode step; state_slots int32 [sequences].
+cosmos::StepRows step_rows(const OptT& portions, const OptT& lens, const Tensor& state_slots, int64_t n_rows, int64_t n_state_slots) {
+  cosmos::StepRows r;
+  check_i32(state_slots, "state_slots");
+  r.state_slots = state_slots.data_ptr<int>();
+  r.n_state_slots = (int)n_state_slots;
+  if (has(portions)) {
+    check_i32(*portions, "portions");
+    TORCH_CHECK(portions->dim() == 2 && portions->size(1) == 4, "portions must be [p, 4]");
+    r.portions = portions->data_ptr(); r.n = (int)portions->size(0);
+  } else {
+    TORCH_CHECK(has(lens), "a decode step needs lens");
+    check_i32(*lens, "lens");
+    TORCH_CHECK(lens->numel() == n_rows && state_slots.numel() == n_rows, "one row per sequence");
+    r.lens = lens->data_ptr<int>(); r.n = (int)n_rows;
+  }
+  return r;
+}
+Tensor padded_rows(int64_t n, int64_t cols, const at::TensorOptions& o) {
+  return at::empty({n, (cols + 7) / 8 * 8}, o).narrow(1, 0, cols);
+}
+
+// See BranchNormArgs. x [n, d] fp32 in place; `normed` up to two branches with their weights; h1 / h2 [n, >= d].
+void branch_norm_(Tensor x, const OptT& embed, const OptT& tokens, double embed_scale, const OptT& pos_turns, const OptT& positions,
+                  at::TensorList normed, at::TensorList normed_w, double coef, const OptT& plain, const OptT& gamma1, const OptT& gamma2,
+                  double gamma_add, double eps, const OptT& h1, const OptT& h2, bool f32) {
+  TORCH_CHECK(x.is_cuda() && x.scalar_type() == at::kFloat && x.dim() == 2 && x.is_contiguous(), "x must be fp32 [n, d]");
+  c10::cuda::CUDAGuard guard(x.device());
+  cosmos::BranchNormArgs a;
+  const int64_t n = x.size(0), d = x.size(1);
+  a.x = x.data_ptr<float>(); a.rows = n; a.d = (int)d; a.is_f32 = f32;
+  a.status = status_ptr(x);
+  if (has(embed)) {
+    TORCH_CHECK(has(tokens) && tokens->numel() == n && embed->dim() == 2 && embed->size(1) == d && embed->stride(1) == 1 &&
+                is_f32(*embed, "embed") == f32);
+    a.embed = embed->data_ptr(); a.ld_embed = embed->stride(0); a.vocab = (int)embed->size(0);
+    a.tokens = i64_ptr(*tokens, "tokens"); a.embed_scale = (float)embed_scale;
+    if (has(pos_turns)) {
+      TORCH_CHECK(pos_turns->is_cuda() && pos_turns->scalar_type() == at::kDouble && pos_turns->is_contiguous() &&
+                      pos_turns->numel() == (d + 1) / 2 && has(positions) && positions->numel() == n, "bad position table");
+      a.pos_turns = pos_turns->data_ptr<double>();
+      a.positions = i64_ptr(*positions, "positions");
+    }
+  }
+  TORCH_CHECK(normed.size() <= 2 && normed.size() == normed_w.size(), "up to two normed branches with a weight each");
+  a.n_normed = (int)normed.size(); a.coef = (float)coef;
+  for (size_t i = 0; i < normed.size(); ++i) {
+    a.normed[i] = row_source(normed[i], f32, n, d, "branch");
+    a.normed_w[i] = f32_vec(normed_w[i], d, "branch weight");
+  }
+  if (has(plain)) {
+    a.has_plain = true;
+    a.plain = row_source(*plain, f32, n, d, "plain");
+  }
+  const OptT* hs[2] = {&h1, &h2};
+  const OptT* gs[2] = {&gamma1, &gamma2};
+  for (int i = 0; i < 2; ++i) {
+    if (!has(*hs[i])) continue;
+    const Tensor& h = **hs[i];
+    TORCH_CHECK(has(*gs[i]) && is_f32(h, "h") == f32 && h.dim() == 2 && h.size(0) >= n && h.size(1) >= d && h.stride(1) == 1, "bad h");
+    TORCH_CHECK(a.ldh == 0 || a.ldh == h.stride(0), "h1 and h2 must have one row stride");
+    a.h[i] = h.data_ptr(); a.ldh = h.stride(0);
+    a.gamma[i] = f32_vec(**gs[i], d, "gamma");
+  }
+  a.gamma_add = (float)gamma_add; a.eps = (float)eps;
+  cosmos::branch_norm(a, cur_stream());
+}
+
+// See QkNormArgs -> q [n, H, dim]
+Tensor qk_norm_post(const Tensor& q, const Tensor& k, int64_t H, int64_t G, const Tensor& wq, const Tensor& wk, double eps,
+                    double temp_coef, int64_t temp_every, const Tensor& positions, const Tensor& slots, Tensor k_cache, Tensor v_cache) {
+  c10::cuda::CUDAGuard guard(q.device());
+  cosmos::QkNormArgs a;
+  a.is_f32 = is_f32(k_cache, "k_cache");
+  TORCH_CHECK(k_cache.dim() == 4 && k_cache.is_contiguous() && v_cache.is_contiguous() && v_cache.sizes() == k_cache.sizes() &&
+                  v_cache.scalar_type() == k_cache.scalar_type() && k_cache.size(1) == G, "caches must be contiguous [pages, G, page_size, dim]");
+  a.n = slots.numel(); a.H = (int)H; a.G = (int)G; a.dim = (int)k_cache.size(3);
+  a.q = row_source(q, a.is_f32, a.n, H * a.dim, "q");
+  a.k = row_source(k, a.is_f32, a.n, G * a.dim, "k");
+  a.wq = f32_vec(wq, H * a.dim, "wq"); a.wk = f32_vec(wk, G * a.dim, "wk");
+  a.eps = (float)eps; a.temp_coef = (float)temp_coef; a.temp_every = temp_every;
+  TORCH_CHECK(positions.numel() == a.n, "one position per token");
+  a.positions = i64_ptr(positions, "positions"); a.slots = i64_ptr(slots, "slots");
+  a.n_slots = k_cache.size(0) * k_cache.size(2); a.page_size = (int)k_cache.size(2);
+  a.k_cache = k_cache.data_ptr(); a.v_cache = v_cache.data_ptr();
+  Tensor out = at::empty({a.n, H, a.dim}, k_cache.options());
+  a.q_out = out.data_ptr();
+  a.status = status_ptr(k_cache);
+  cosmos::qk_norm_post(a, cur_stream());
+  return out;
+}
+
+// See CausalConvArgs -> u [n, inner] (row stride padded to 8)
+Tensor causal_conv(const Tensor& x, const Tensor& w, const Tensor& b, Tensor conv_state, const Tensor& state_slots,
+                   const OptT& portions, const OptT& tiles, const OptT& lens, int64_t n) {
+  c10::cuda::CUDAGuard guard(x.device());
+  cosmos::CausalConvArgs a;
+  TORCH_CHECK(w.dim() == 2 && conv_state.dim() == 3 && conv_state.is_contiguous() && conv_state.size(1) == w.size(1) - 1 &&
+                  conv_state.size(2) == w.size(0), "conv_state must be [slots, taps - 1, inner]");
+  a.is_f32 = is_f32(conv_state, "conv_state");
+  a.inner = (int)w.size(0); a.taps = (int)w.size(1);
+  a.x = row_source(x, a.is_f32, n, a.inner, "x");
+  a.w = f32_vec(w, w.numel(), "w"); a.b = f32_vec(b, a.inner, "b");
+  a.conv_state = conv_state.data_ptr();
+  a.rows = step_rows(portions, lens, state_slots, n, conv_state.size(0));
+  if (has(portions)) {
+    TORCH_CHECK(has(tiles), "portions need their tiles");
+    check_i32(*tiles, "tiles");
+    TORCH_CHECK(tiles->dim() == 2 && tiles->size(1) == 8, "tiles must be [t, 8]");
+    a.tiles = tiles->data_ptr<int>(); a.n_tiles = (int)tiles->size(0);
+  }
+  Tensor u = padded_rows(n, a.inner, conv_state.options());
+  a.u = u.data_ptr(); a.ldu = u.stride(0);
+  a.status = status_ptr(x);
+  cosmos::causal_conv(a, cur_stream());
+  return u;
+}
+
+// See SelectiveScanArgs. y [n, >= inner]: columns [0, inner) are written, and zeros into [inner, y_cols).
+void selective_scan(const Tensor& u, const Tensor& dt, const Tensor& z, const Tensor& bc, const Tensor& dt_bias, const Tensor& a2,
+                    const Tensor& D, Tensor S, Tensor y, int64_t y_cols, const Tensor& state_slots, const OptT& portions,
+                    const OptT& lens) {
+  c10::cuda::CUDAGuard guard(u.device());
+  cosmos::SelectiveScanArgs a;
+  a.is_f32 = is_f32(u, "u");
+  const int64_t n = u.size(0);
+  TORCH_CHECK(S.dim() == 3 && S.scalar_type() == at::kFloat && S.is_contiguous(), "S must be fp32 [slots, inner, state]");
+  a.inner = (int)S.size(1); a.state = (int)S.size(2);
+  TORCH_CHECK(u.dim() == 2 && u.size(1) == a.inner && u.stride(1) == 1 && is_f32(y, "y") == a.is_f32 && y.dim() == 2 &&
+                  y.size(0) == n && y.stride(1) == 1 && y.size(1) >= y_cols && y_cols >= a.inner, "bad u or y");
+  a.u = u.data_ptr(); a.ldu = u.stride(0);
+  a.dt = row_source(dt, a.is_f32, n, a.inner, "dt");
+  a.z = row_source(z, a.is_f32, n, a.inner, "z");
+  a.bc = row_source(bc, a.is_f32, n, 2 * a.state, "bc");
+  a.dt_bias = f32_vec(dt_bias, a.inner, "dt_bias");
+  a.a2 = f32_vec(a2, (int64_t)a.inner * a.state, "a2");
+  a.D = f32_vec(D, a.inner, "D");
+  a.S = S.data_ptr<float>();
+  a.y = y.data_ptr(); a.ldy = y.stride(0);
+  a.rows = step_rows(portions, lens, state_slots, n, S.size(0));
+  a.status = status_ptr(u);
+  cosmos::selective_scan(a, cur_stream());
+  cosmos::zero_cols(a.y, a.ldy, a.inner, (int)y_cols, n, a.is_f32, cur_stream());
+}
+
+// See MatrixMemoryArgs -> o [n, H * vdim] (row stride padded to 8). S [slots, H, dim, vdim], nrm [slots, H, slices, dim],
+// m [slots, H, slices] fp32.
+Tensor matrix_memory(const Tensor& q, const Tensor& k, const Tensor& v, const Tensor& gates, const Tensor& gate_bias, double q_scale,
+                     double cap, Tensor S, Tensor nrm, Tensor m, const Tensor& state_slots, const OptT& portions, const OptT& lens,
+                     int64_t n, bool f32) {
+  c10::cuda::CUDAGuard guard(q.device());
+  cosmos::MatrixMemoryArgs a;
+  TORCH_CHECK(S.dim() == 4 && S.scalar_type() == at::kFloat && S.is_contiguous(), "S must be fp32 [slots, H, dim, vdim]");
+  a.is_f32 = f32;
+  a.H = (int)S.size(1); a.dim = (int)S.size(2); a.vdim = (int)S.size(3);
+  const int64_t slices = (a.vdim + cosmos::MEMORY_SLICE - 1) / cosmos::MEMORY_SLICE;
+  a.S = S.data_ptr<float>();
+  a.n = const_cast<float*>(f32_vec(nrm, S.size(0) * a.H * slices * a.dim, "nrm"));
+  a.m = const_cast<float*>(f32_vec(m, S.size(0) * a.H * slices, "m"));
+  a.q = row_source(q, f32, n, (int64_t)a.H * a.dim, "q");
+  a.k = row_source(k, f32, n, (int64_t)a.H * a.dim, "k");
+  a.v = row_source(v, f32, n, (int64_t)a.H * a.vdim, "v");
+  TORCH_CHECK(gates.scalar_type() == at::kFloat, "gates must be fp32");
+  a.gates = row_source(gates, true, n, 2 * a.H, "gates");
+  a.gate_bias = f32_vec(gate_bias, 2 * a.H, "gate_bias");
+  a.q_scale = (float)q_scale; a.cap = (float)cap;
+  a.rows = step_rows(portions, lens, state_slots, n, S.size(0));
+  Tensor o = padded_rows(n, (int64_t)a.H * a.vdim, S.options().dtype(f32 ? at::kFloat : at::kBFloat16));
+  a.o = o.data_ptr(); a.ldo = o.stride(0);
+  a.status = status_ptr(q);
+  cosmos::matrix_memory(a, cur_stream());
+  return o;
+}
+
+// y = o / rms(head of o) * w * sigmoid(g), heads of w.numel() / H columns
+Tensor head_norm_gate(const Tensor& o, const Tensor& g, const Tensor& w, int64_t H, double eps) {
+  c10::cuda::CUDAGuard guard(o.device());
+  cosmos::HeadNormGateArgs a;
+  a.is_f32 = is_f32(o, "o");
+  const int64_t cols = w.numel();
+  TORCH_CHECK(o.dim() == 2 && o.size(1) == cols && o.stride(1) == 1 && H > 0 && cols % H == 0, "o must be [n, H * vdim]");
+  a.o = o.data_ptr(); a.ldo = o.stride(0); a.n = o.size(0); a.H = (int)H; a.vdim = (int)(cols / H);
+  a.g = row_source(g, a.is_f32, a.n, cols, "g");
+  a.w = f32_vec(w, cols, "w"); a.eps = (float)eps;
+  Tensor y = padded_rows(a.n, cols, o.options());
+  a.y = y.data_ptr(); a.ldy = y.stride(0);
+  cosmos::head_norm_gate(a, cur_stream());
+  return y;
+}
+
 }  // namespace
 
 TORCH_LIBRARY_FRAGMENT(cosmos_b200, m) {
@@ -303,4 +515,10 @@ TORCH_LIBRARY_FRAGMENT(cosmos_b200, m) {
   m.def("moe_route", &moe_route);
   m.def("grouped_gemm", &grouped_gemm);
   m.def("gemm_partial", &gemm_partial);
+  m.def("branch_norm_", &branch_norm_);
+  m.def("qk_norm_post", &qk_norm_post);
+  m.def("causal_conv", &causal_conv);
+  m.def("selective_scan", &selective_scan);
+  m.def("matrix_memory", &matrix_memory);
+  m.def("head_norm_gate", &head_norm_gate);
 }

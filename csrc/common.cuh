@@ -51,6 +51,7 @@ enum : int {
   SITE_STACK_PAGE = 7,    // page id read by windowed attention
   SITE_MOE_EXPERT = 8,    // expert id of a routing table
   SITE_MOE_ROW = 9,       // row of the expert-sorted buffers
+  SITE_STATE_SLOT = 10,   // recurrent-state slot of a layer stack's step
   SITE_SELFTEST = 15,
 };
 

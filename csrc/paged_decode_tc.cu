@@ -101,7 +101,7 @@ __device__ __forceinline__ bool pt_bar_all_ok(bool ok) {
 struct PtWin {
   int window, kdim, vdim;
   const float* r1;   // [Hq]; null = no bias
-  const float* r2;
+  const float* r2;   // null = linear bias
   long long ldq, ldo;
 };
 
@@ -341,8 +341,8 @@ paged_decode_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_con
 #pragma unroll
       for (int g = 0; g < GROUP; ++g) {
         m_used[g] = -1e30f; l_part[g] = 0.f;
-        b1[g] = WIN && win.r1 ? win.r1[I.kvh * GROUP + g] : 0.f;
-        b2[g] = WIN && win.r1 ? win.r2[I.kvh * GROUP + g] : 0.f;
+        b1[g] = WIN && win.r1 ? win.r1[I.kvh * GROUP + g] * (win.r2 ? 1.f : 1.4426950408889634f) : 0.f;
+        b2[g] = WIN && win.r2 ? win.r2[I.kvh * GROUP + g] : 0.f;
       }
       for (int j = 0; j < I.n_tiles; ++j, ++gt) {
         ok = ok && mbar_wait(B(PB_S + (gt & 1)), (gt >> 1) & 1, abort_flag, status, ST_TIMEOUT_SOFTMAX);
@@ -359,7 +359,7 @@ paged_decode_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_con
 #pragma unroll
         for (int g = 0; g < GROUP; ++g) {
           x[g] = __uint_as_float(sv[g]) * scale_log2;
-          if (WIN) x[g] -= b1[g] * __log2f(fmaf(b2[g], (float)dist, 1.f));
+          if (WIN) x[g] -= b1[g] * (win.r2 ? __log2f(fmaf(b2[g], (float)dist, 1.f)) : (float)dist);
           x[g] = valid ? x[g] : -1e30f;
           float v = x[g];
 #pragma unroll

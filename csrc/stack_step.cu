@@ -5,77 +5,9 @@
 #include "common.cuh"
 #include "launch.cuh"
 #include "stack.h"
+#include "vec.cuh"
 
 namespace cb {
-
-template <typename T> struct Elem;
-template <> struct Elem<float> {
-  static __device__ __forceinline__ float get(const float* p) { return *p; }
-  static __device__ __forceinline__ void put(float* p, float v) { *p = v; }
-};
-template <> struct Elem<bf16> {
-  static __device__ __forceinline__ float get(const bf16* p) { return __bfloat162float(*p); }
-  static __device__ __forceinline__ void put(bf16* p, float v) { *p = __float2bfloat16(v); }
-};
-template <typename T, int VEC> struct Vec {
-  static __device__ __forceinline__ void load(const T* p, float (&v)[VEC]) {
-#pragma unroll
-    for (int e = 0; e < VEC; ++e) v[e] = Elem<T>::get(p + e);
-  }
-  static __device__ __forceinline__ void store(T* p, const float (&v)[VEC]) {
-#pragma unroll
-    for (int e = 0; e < VEC; ++e) Elem<T>::put(p + e, v[e]);
-  }
-};
-template <> struct Vec<float, 4> {
-  static __device__ __forceinline__ void load(const float* p, float (&v)[4]) {
-    const float4 x = *reinterpret_cast<const float4*>(p);
-    v[0] = x.x; v[1] = x.y; v[2] = x.z; v[3] = x.w;
-  }
-  static __device__ __forceinline__ void store(float* p, const float (&v)[4]) {
-    *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
-  }
-};
-template <> struct Vec<bf16, 4> {
-  static __device__ __forceinline__ void load(const bf16* p, float (&v)[4]) {
-    const uint2 x = *reinterpret_cast<const uint2*>(p);
-    v[0] = bf16lo(x.x); v[1] = bf16hi(x.x); v[2] = bf16lo(x.y); v[3] = bf16hi(x.y);
-  }
-  static __device__ __forceinline__ void store(bf16* p, const float (&v)[4]) {
-    uint2 o;
-    o.x = pack_bf16(v[0], v[1]); o.y = pack_bf16(v[2], v[3]);
-    *reinterpret_cast<uint2*>(p) = o;
-  }
-};
-
-template <> struct Vec<float, 8> {
-  static __device__ __forceinline__ void load(const float* p, float (&v)[8]) {
-    const float4 x = reinterpret_cast<const float4*>(p)[0], y = reinterpret_cast<const float4*>(p)[1];
-    v[0] = x.x; v[1] = x.y; v[2] = x.z; v[3] = x.w; v[4] = y.x; v[5] = y.y; v[6] = y.z; v[7] = y.w;
-  }
-  static __device__ __forceinline__ void store(float* p, const float (&v)[8]) {
-    reinterpret_cast<float4*>(p)[0] = make_float4(v[0], v[1], v[2], v[3]);
-    reinterpret_cast<float4*>(p)[1] = make_float4(v[4], v[5], v[6], v[7]);
-  }
-};
-template <> struct Vec<bf16, 8> {
-  static __device__ __forceinline__ void load(const bf16* p, float (&v)[8]) {
-    const uint4 x = *reinterpret_cast<const uint4*>(p);
-    v[0] = bf16lo(x.x); v[1] = bf16hi(x.x); v[2] = bf16lo(x.y); v[3] = bf16hi(x.y);
-    v[4] = bf16lo(x.z); v[5] = bf16hi(x.z); v[6] = bf16lo(x.w); v[7] = bf16hi(x.w);
-  }
-  static __device__ __forceinline__ void store(bf16* p, const float (&v)[8]) {
-    uint4 o;
-    o.x = pack_bf16(v[0], v[1]); o.y = pack_bf16(v[2], v[3]); o.z = pack_bf16(v[4], v[5]); o.w = pack_bf16(v[6], v[7]);
-    *reinterpret_cast<uint4*>(p) = o;
-  }
-};
-
-__device__ __forceinline__ float warp_add(float v) {
-#pragma unroll
-  for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
-  return v;
-}
 
 // The common case of residual_norm_kernel (below), tuned for whole prompts: at most 4 vectors of 8 per thread, kept in
 // registers (all loads of a row are issued before the first use), one or two parts of at least a warp's vectors each.

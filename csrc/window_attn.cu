@@ -53,7 +53,7 @@ window_attn_simt_kernel(const cosmos::WindowAttnArgs a) {
     qs[i] = r < rows ? ws_get(q + (long long)r * a.ldq + c) : 0.f;
   }
   for (int i = tid; i < WS_ROWS * vdim; i += WS_THREADS) os[i] = 0.f;
-  const float r1 = a.r1 ? a.r1[h] : 0.f, r2 = a.r1 ? a.r2[h] : 0.f;
+  const float r1 = a.r1 ? a.r1[h] : 0.f, r2 = a.r2 ? a.r2[h] : 0.f;
   float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};
   const int lo = max(0, pos0 - a.window + 1), hi = pos0 + rows;
   for (int k0 = lo; k0 < hi; k0 += WS_KEYS) {
@@ -82,7 +82,7 @@ window_attn_simt_kernel(const cosmos::WindowAttnArgs a) {
         float dot = 0.f;
         for (int c = 0; c < dim; ++c) dot = fmaf(qs[r * dim + c], ks[lane * (dim + 1) + c], dot);
         s = dot * a.scale;
-        if (a.r1) s -= r1 * log1pf(r2 * (float)dist);
+        if (a.r1) s -= r1 * (a.r2 ? log1pf(r2 * (float)dist) : (float)dist);
       }
       float mx = s;
 #pragma unroll

@@ -8,7 +8,7 @@
 //     sequences. Only the key blocks inside [first row's window, last row] are visited, and each 128-row tile skips those
 //     of them that lie outside its own rows' range.
 //   * Mask and bias are one table. Within a 128 x 128 block the distance i - j takes 255 values, so the softmax warps of a
-//     tile compute bias[i - j] once per block (two logarithms per thread), with -inf outside the window and above the
+//     tile compute bias[i - j] once per block (at most two logarithms per thread), with -inf outside the window and above the
 //     diagonal, and add it with the FMA that scales the scores. A row's entries are consecutive; four copies of the table,
 //     each shifted by one entry, let every thread read four at a time with aligned 16-byte loads. The copies start 8 words
 //     apart modulo the 32 banks, so the eight lanes of a 16-byte load phase hit different banks. Half of a row's entries
@@ -275,7 +275,8 @@ window_attn_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
     const uint32_t s_addr = lane_addr + t * 128;
     const uint32_t o_addr = lane_addr + 256 + t * 128;
     const float sl2 = p.scale_log2;
-    const float r1 = p.r1 ? p.r1[head] : 0.f, r2 = p.r1 ? p.r2[head] : 0.f;
+    const bool linear = p.r2 == nullptr;   // scores are in base 2
+    const float r1 = p.r1 ? p.r1[head] * (linear ? 1.4426950408889634f : 1.f) : 0.f, r2 = linear ? 0.f : p.r2[head];
     // table entry u = column - row + 127 stands for the distance d0 - (u - 127), d0 = distance of (row 0, column 0)
     const int shift = (127 - row) & 3;
     float* tab_t = reinterpret_cast<float*>(gen + WA_OFF_TAB + t * 2 * WA_TAB_BYTES);
@@ -289,7 +290,7 @@ window_attn_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid
       for (int e = 0; e < 2; ++e) {
         const int u = row + 128 * e;
         const int dist = d0 - (u - 127);
-        const float b = (dist >= 0 && dist < p.window) ? -r1 * __log2f(fmaf(r2, (float)dist, 1.f)) : -INFINITY;
+        const float b = (dist >= 0 && dist < p.window) ? -r1 * (linear ? (float)dist : __log2f(fmaf(r2, (float)dist, 1.f))) : -INFINITY;
 #pragma unroll
         for (int c = 0; c < 4; ++c)
           if (u >= c) tab[c * WA_TAB + u - c] = b;   // copy c: entry i holds table entry i + c
