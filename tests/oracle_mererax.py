@@ -206,11 +206,14 @@ def random_tensors(cfg, seed, std=None):
             out[p + "mix.left.q.norm"], out[p + "mix.left.k.norm"] = 1 + rnd(q, scale=0.2), 1 + rnd(k, scale=0.2)
             out[p + "mix.left.o"] = mat(d, a["heads"] * a["vdim"])
             hd, hv = r["heads"] * r["dim"], r["heads"] * r["vdim"]
-            out[p + "mix.right.q"], out[p + "mix.right.k"] = mat(hd, d), mat(hd, d)
+            # queries and keys lean the same way: a q . k near zero flips the sign of a young memory's normed output, and
+            # 16-bit rounding would then decide it
+            out[p + "mix.right.q"] = mat(hd, d)
+            out[p + "mix.right.k"] = 0.85 * out[p + "mix.right.q"] + mat(hd, d, 0.5)
             out[p + "mix.right.v"], out[p + "mix.right.g"] = mat(hv, d), mat(hv, d)
             out[p + "mix.right.o"], out[p + "mix.right.norm"] = mat(d, hv), 1 + rnd(hv, scale=0.2)
             out[p + "mix.right.i"], out[p + "mix.right.f"] = mat(r["heads"], d), mat(r["heads"], d)
-            out[p + "mix.right.i.b"], out[p + "mix.right.f.b"] = rnd(r["heads"]), rnd(r["heads"]) + 3.0
+            out[p + "mix.right.i.b"], out[p + "mix.right.f.b"] = rnd(r["heads"]) - 2.0, rnd(r["heads"]) + 2.0
             out[p + "mix.left.out"], out[p + "mix.right.out"] = 1 + rnd(d, scale=0.2), 1 + rnd(d, scale=0.2)
         if layer.get("mlp") is not None:
             ff = layer["mlp"]["ff"]
