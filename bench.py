@@ -27,7 +27,8 @@ sample, under `extra`:
 A phase that fails or runs out of its time budget is reported as an error string and does not affect the
 headline. `--no-extras` skips them.
 
-`--workload stack` measures something else instead: the decoder stacks (models/stack.py), see that option's help.
+`--workload stack` and `--workload mererax` measure something else instead: the decoder stacks (models/stack.py), see that
+option's help.
 
 `--impl library`: the same model, layout and sampler with every op on PyTorch's library kernels (cuBLAS,
 fused SDPA, eager element-wise) and NCCL collectives instead of this package's kernels: the A/B arm.
@@ -419,21 +420,22 @@ def phase_train(c: Ctx, rec: dict):
 
 
 def stack_workload(c: Ctx) -> int:
-    """`--workload stack`: one line with the decoder-stack numbers (cosmos_b200/serve/bench_stack.py)."""
-    from cosmos_b200.serve import bench_stack
+    """`--workload stack` / `mererax`: one line with the decoder-stack numbers (cosmos_b200/serve/bench_stack.py, bench_mererax.py)."""
+    from cosmos_b200.serve import bench_mererax, bench_stack
 
     if c.world > 1:
-        raise SystemExit("--workload stack runs on one GPU")
+        raise SystemExit(f"--workload {c.args.workload} runs on one GPU")
+    design, bench = ("Lederax", bench_stack) if c.args.workload == "stack" else ("Mererax", bench_mererax)
     from cosmos_b200 import ops
     _, hbm, src = _peaks()
     p = os.path.join(os.path.dirname(os.path.abspath(__file__)), "MEASURED_PEAKS.json")
     burst = json.load(open(p))["bf16_tflops"] if src == "measured" else 1590.0
     smp = c.sampler()
     l0 = ops.launch_count()
-    res = bench_stack.run(max(c.args.steps, 20), burst, hbm)
+    res = bench.run(max(c.args.steps, 20), burst, hbm)
     clocks = smp.stop()
     first = res["throughput"]["d4096"]
-    print(json.dumps({"metric": "decoder_stack_prefill_tokens_per_s (Lederax layers, d 4096, 16384-token prompt)",
+    print(json.dumps({"metric": f"decoder_stack_prefill_tokens_per_s ({design} layers, d 4096, 16384-token prompt)",
                       "value": first["prefill"]["tokens_per_s"], "unit": "tokens/s", "n_gpus": 1, "higher_is_better": True,
                       "dtype": "bf16", "data": "synthetic (random token ids, random-init weights)",
                       "peaks": {"source": src, "bf16_tflops": burst, "hbm_gbs": hbm}, "gpu_launches": ops.launch_count() - l0,
@@ -459,9 +461,10 @@ def main():
     ap.add_argument("--cfgp-size", type=int, default=0, help="explicit layout: CFG parallel (1 or 2)")
     ap.add_argument("--cp-mode", default="ulysses", choices=["ulysses", "ring"])
     ap.add_argument("--no-extras", action="store_true", help="headline only (no s/video, decode, training phases)")
-    ap.add_argument("--workload", default="dit", choices=["dit", "stack"],
+    ap.add_argument("--workload", default="dit", choices=["dit", "stack", "mererax"],
                     help="dit: the headline above (default); stack: prefill / decode throughput and kernel times of a decoder "
-                         "stack (Lederax layers, random weights) beside the Reasoner's tower at equal size, one GPU")
+                         "stack (Lederax layers, random weights) beside the Reasoner's tower at equal size, one GPU; mererax: the "
+                         "same for Mererax layers")
     ap.add_argument("--extras", default="video,decode,train", help="which extra phases to run")
     ap.add_argument("--extras-budget-s", type=float, default=330.0,
                     help="a phase is not started once the extras have used this much wall time")
@@ -484,7 +487,7 @@ def main():
         raise SystemExit("cosmos_b200 kernel library failed to load")
     if c.library:
         ops.set_backend("library")
-    if args.workload == "stack":
+    if args.workload != "dit":
         return stack_workload(c)
     rec: dict = {}
     phase_dit(c, rec)
