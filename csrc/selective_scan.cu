@@ -1,10 +1,10 @@
 // Selective scan (stack.h): causal convolution with its state, the scan over portions of prompts, and the decode step.
 //
-// Scan over a portion: a CTA owns CH channels of one portion, four lanes a channel, NS of its states per lane in registers for
-// the whole portion. Tokens come in tiles of 16: the next tile's rows are loaded into registers while the current one is
-// worked on, and softplus, dt * u and the gate silu(z) are computed once per (token, channel) on the way to shared memory.
-// What is left per (token, channel, state) is one exponential and four multiply-adds; the sums over a channel's four lanes
-// are reduced for four tokens at a time (three exchanges), after which each lane finishes one token.
+// Scan over a portion: a CTA owns CH channels of one portion. Half of its warps scan: four lanes a channel, NS of its states per
+// lane in registers for the whole portion, one exponential and two packed pairs of multiply-adds per state and token; the sums
+// over a channel's four lanes are reduced for four tokens at a time (three exchanges), after which each lane holds one token's.
+// The other warps feed them: they load the next tile of 32 tokens, compute softplus, dt * u and the gate silu(z) once per (token,
+// channel), and write out the finished tile before the current one. The two halves meet once per tile.
 #include <algorithm>
 #include <stdexcept>
 
@@ -15,7 +15,66 @@
 
 namespace cb {
 
+__device__ __forceinline__ float silu_fast(float z) { return __fdividef(z, 1.f + fast_ex2(-1.4426950408889634f * fmaxf(z, -80.f))); }
+
 // ------------------------------------------------------------------ causal convolution
+// Rows of finished values, 8 channels per thread: the loads of the next rows are in flight while one is worked on.
+template <typename T, int TAPS>
+__global__ void __launch_bounds__(128)
+causal_conv_rows_kernel(const cosmos::CausalConvArgs a) {
+  const int c = (blockIdx.x * blockDim.x + threadIdx.x) * 8;
+  if (c >= a.inner) return;
+  const int* tile = a.tiles + (long long)blockIdx.y * 8;
+  const int seq = tile[0], row0 = tile[1], rows = tile[2], pos0 = tile[3], first = tile[4];
+  const long long slot = get_state_slot(a.rows, seq, a.status);
+  if (slot < 0) return;
+  const T* x = reinterpret_cast<const T*>(a.x.p) + c;
+  const T* st = reinterpret_cast<const T*>(a.conv_state) + slot * (TAPS - 1) * a.inner + c;
+  T* u = reinterpret_cast<T*>(a.u) + c;
+  constexpr int AHEAD = 8, H = TAPS > 1 ? TAPS - 1 : 1;
+  Raw<T, 8> nx[AHEAD];
+#pragma unroll
+  for (int i = 0; i < AHEAD; ++i) nx[i].load(x + (long long)(row0 + min(i, rows - 1)) * a.x.ld);
+  float hist[H][8], w[TAPS][8], bias[8];
+#pragma unroll
+  for (int j = 0; j < TAPS - 1; ++j) {
+    const int src = row0 - (TAPS - 1) + j;
+    if (src >= first) {
+      Vec<T, 8>::load(x + (long long)src * a.x.ld, hist[j]);
+    } else if (pos0 > 0) {
+      Vec<T, 8>::load(st + (long long)(TAPS - 1 + src - first) * a.inner, hist[j]);
+    } else {
+#pragma unroll
+      for (int e = 0; e < 8; ++e) hist[j][e] = 0.f;
+    }
+  }
+  Vec<float, 8>::load(a.b + c, bias);
+#pragma unroll
+  for (int e = 0; e < 8; ++e)
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) w[j][e] = a.w[(long long)(c + e) * TAPS + j];
+  for (int r8 = 0; r8 < rows; r8 += AHEAD) {
+#pragma unroll
+    for (int i = 0; i < AHEAD; ++i) {
+      const int r = r8 + i;
+      float v[8], s[8];
+      nx[i].get(v);
+      nx[i].load(x + (long long)(row0 + min(r + AHEAD, rows - 1)) * a.x.ld);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) {
+        s[e] = bias[e];
+#pragma unroll
+        for (int j = 0; j < TAPS - 1; ++j) s[e] = fmaf(w[j][e], hist[j][e], s[e]);
+        s[e] = silu_fast(fmaf(w[TAPS - 1][e], v[e], s[e]));
+#pragma unroll
+        for (int j = 0; j + 1 < TAPS - 1; ++j) hist[j][e] = hist[j + 1][e];
+        hist[H - 1][e] = v[e];
+      }
+      if (r < rows) Vec<T, 8>::store(u + (long long)(row0 + r) * a.ldu, s);
+    }
+  }
+}
+
 // grid (channel blocks, tiles or sequences). A decode step updates the conv state here (a thread owns its channels); portions do
 // it in conv_state_kernel, because another tile of the portion may still read the old state.
 template <typename T, int VEC, int TAPS>   // TAPS 0: any number up to CONV_MAX_TAPS
@@ -87,7 +146,7 @@ causal_conv_kernel(const cosmos::CausalConvArgs a) {
 #pragma unroll
     for (int e = 0; e < VEC; ++e) {
       const float wl = TAPS ? w[TAPS ? TAPS - 1 : 0][e] : a.w[(long long)(c + e) * taps + taps - 1];
-      s[e] = silu_f32(fmaf(wl, x[e], s[e]));
+      s[e] = silu_fast(fmaf(wl, x[e], s[e]));
     }
     Vec<T, VEC>::store(u + (long long)(row0 + r) * a.ldu + c, s);
 #pragma unroll
@@ -142,137 +201,246 @@ conv_state_kernel(const cosmos::CausalConvArgs a) {
 }
 
 // ------------------------------------------------------------------ scan
-__device__ __forceinline__ float softplus_f32(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
+// log(1 + e^x) for the step sizes: max(x, 0) + log(1 + e) with e = e^-|x|, and log(1 + e) = 2 atanh(s), s = e / (2 + e) <= 1/3,
+// by the series of atanh, which keeps the digits of a small e.
+__device__ __forceinline__ float softplus_f32(float x) {
+  const float e = fast_ex2(-1.4426950408889634f * fabsf(x));
+  const float s = __fdividef(e, 2.f + e), q = s * s;
+  float r = fmaf(q, 1.f / 13.f, 1.f / 11.f);
+  r = fmaf(q, r, 1.f / 9.f);
+  r = fmaf(q, r, 1.f / 7.f);
+  r = fmaf(q, r, 1.f / 5.f);
+  r = fmaf(q, r, 1.f / 3.f);
+  r = fmaf(q, r, 1.f);
+  return fmaf(2.f * s, r, fmaxf(x, 0.f));
+}
 
-constexpr int SC_TT = 16;   // tokens per tile
+__device__ __forceinline__ uint64_t pack2(float lo, float hi) {
+  uint64_t r;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(lo), "f"(hi));
+  return r;
+}
+__device__ __forceinline__ float2 unpack2(uint64_t v) {
+  float2 r;
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(r.x), "=f"(r.y) : "l"(v));
+  return r;
+}
+__device__ __forceinline__ uint64_t mul2(uint64_t a, uint64_t b) {
+  uint64_t r;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+  return r;
+}
+__device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
+  uint64_t r;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+  return r;
+}
 
-template <typename T, int NS, int CH>
-__global__ void __launch_bounds__(4 * CH)
+// NP pairs from shared memory
+template <int NP>
+__device__ __forceinline__ void load_pairs(const float* p, uint64_t (&v)[NP]) {
+  if constexpr (NP % 2 == 0) {
+#pragma unroll
+    for (int i = 0; i < NP; i += 2) {
+      const ulonglong2 x = *reinterpret_cast<const ulonglong2*>(p + 2 * i);
+      v[i] = x.x; v[i + 1] = x.y;
+    }
+  } else {
+#pragma unroll
+    for (int i = 0; i < NP; ++i) v[i] = *reinterpret_cast<const unsigned long long*>(p + 2 * i);
+  }
+}
+
+constexpr int SC_TT = 32;   // tokens per tile
+
+// The two halves of the CTA meet here from different places in the code.
+template <int N>
+__device__ __forceinline__ void tile_barrier() {
+  asm volatile("barrier.sync 1, %0;" ::"n"(N) : "memory");
+}
+
+template <int NS, int CH>
+struct ScanSmem {
+  float2 du[2][SC_TT][CH];            // dt, dt * u
+  float2 uz[2][SC_TT][CH];            // u, silu(z); then the finished output in .x
+  float bc[2][SC_TT][2][4 * NS];      // B | C, NS values per lane
+};
+
+// FAST: finished, aligned rows and N = 4 NS, loaded a tile ahead; otherwise rows are loaded when their tile is made.
+template <typename T, int NS, int CH, bool FAST>
+__global__ void __launch_bounds__(8 * CH)
 selective_scan_kernel(const cosmos::SelectiveScanArgs a) {
-  constexpr int NT = 4 * CH, Q = CH / 4;   // threads; groups of four channels
-  static_assert(NT == SC_TT * Q, "a thread loads four channels of one token");
-  __shared__ float2 du_s[2][SC_TT][CH];            // dt, dt * u
-  __shared__ float u_s[2][SC_TT][CH];
-  __shared__ float z_s[2][SC_TT][CH];              // gate, then the finished output
-  __shared__ float bc_s[2][SC_TT][2][4][NS];       // B | C by lane
-  const int tid = threadIdx.x, ch = tid >> 2, lane4 = tid & 3;
+  constexpr int NT = 4 * CH, NP = NS / 2, Q = CH / 4, ROWS = SC_TT * Q / NT;   // threads of a half; a feeder loads ROWS x 4 values
+  static_assert(NS % 2 == 0 && NT % 32 == 0 && ROWS * NT == SC_TT * Q, "tile shape");
+  extern __shared__ __align__(16) uint8_t sm_raw[];
+  ScanSmem<NS, CH>& sm = *reinterpret_cast<ScanSmem<NS, CH>*>(sm_raw);
   const Portion p = get_portion(a.rows, blockIdx.y);
   if (p.rows <= 0) return;
   const long long slot = get_state_slot(a.rows, p.seq, a.status);
   if (slot < 0) return;
-  const int c0 = blockIdx.x * CH, c = c0 + ch, N = a.state;
-  const bool live = c < a.inner;
-  float S[NS], a2[NS];
-  float* sp = a.S + (slot * a.inner + c) * (long long)N + lane4 * NS;
+  const int c0 = blockIdx.x * CH, N = a.state;
+  const int n_tiles = (p.rows + SC_TT - 1) / SC_TT;
+  if (threadIdx.x < NT) {
+    // ---------------- scan
+    const int tid = threadIdx.x, ch = tid >> 2, lane4 = tid & 3, c = c0 + ch;
+    const bool live = c < a.inner;
+    uint64_t S[NP], a2[NP];
+    float* sp = a.S + (slot * a.inner + c) * (long long)N + lane4 * NS;
+    const float* ap = a.a2 + (long long)c * N + lane4 * NS;
 #pragma unroll
-  for (int i = 0; i < NS; ++i) {
-    const bool in = live && lane4 * NS + i < N;
-    S[i] = in && p.pos0 > 0 ? sp[i] : 0.f;
-    a2[i] = in ? a.a2[(long long)c * N + lane4 * NS + i] : 0.f;
-  }
-  const float D = live ? a.D[c] : 0.f;
-  // loader: token lt, channels lc .. lc + 3 of the tile
-  const int lt = tid / Q, lq = (tid % Q) * 4, lc = c0 + lq;
-  float ru[4], rd[4], rz[4], bias[4];
+    for (int i = 0; i < NP; ++i) {
+      const bool i0 = live && lane4 * NS + 2 * i < N, i1 = live && lane4 * NS + 2 * i + 1 < N;
+      S[i] = pack2(i0 && p.pos0 > 0 ? sp[2 * i] : 0.f, i1 && p.pos0 > 0 ? sp[2 * i + 1] : 0.f);
+      a2[i] = pack2(i0 ? ap[2 * i] : 0.f, i1 ? ap[2 * i + 1] : 0.f);
+    }
+    const float D = live ? a.D[c] : 0.f;
+    for (int k = 0; k < n_tiles; ++k) {
+      const int b = k & 1;
+      tile_barrier<8 * CH>();   // tile k is in place
+#pragma unroll 1
+      for (int t4 = 0; t4 < SC_TT; t4 += 4) {
+        float acc[4];
 #pragma unroll
-  for (int e = 0; e < 4; ++e) bias[e] = lc + e < a.inner ? a.dt_bias[lc + e] : 0.f;
-  constexpr int NBC = (SC_TT * 8 * NS + NT - 1) / NT;   // B / C values a thread loads
-  float rbc[NBC];
-  const T* ug = reinterpret_cast<const T*>(a.u);
-  const bool vec = a.inner % 4 == 0 && a.ldu % 4 == 0 && a.dt.ld % 4 == 0 && a.z.ld % 4 == 0 && a.dt.split_stride % 4 == 0 &&
-                   a.z.split_stride % 4 == 0 && (reinterpret_cast<uintptr_t>(a.u) & 15) == 0 &&
-                   (reinterpret_cast<uintptr_t>(a.dt.p) & 15) == 0 && (reinterpret_cast<uintptr_t>(a.z.p) & 15) == 0;
-  auto fetch = [&](int t0) {
-    const int t = t0 + lt;
-    const long long row = p.row0 + t;
-    if (t < p.rows && vec && lc < a.inner) {
-      Vec<T, 4>::load(ug + row * a.ldu + lc, ru);
-      load_source<T, 4>(a.dt, row, lc, rd);
-      load_source<T, 4>(a.z, row, lc, rz);
-    } else {
+        for (int j = 0; j < 4; ++j) {
+          const float2 du = sm.du[b][t4 + j][ch];
+          uint64_t B[NP], C[NP];
+          load_pairs<NP>(&sm.bc[b][t4 + j][0][lane4 * NS], B);
+          load_pairs<NP>(&sm.bc[b][t4 + j][1][lane4 * NS], C);
+          const uint64_t dt2 = pack2(du.x, du.x), x2 = pack2(du.y, du.y);
+          uint64_t s = 0ull;
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const bool in = t < p.rows && lc + e < a.inner;
-        ru[e] = in ? Elem<T>::get(ug + row * a.ldu + lc + e) : 0.f;
-        rd[e] = in ? load_source1<T>(a.dt, row, lc + e) : 0.f;
-        rz[e] = in ? load_source1<T>(a.z, row, lc + e) : 0.f;
+          for (int i = 0; i < NP; ++i) {
+            const float2 e = unpack2(mul2(dt2, a2[i]));
+            S[i] = fma2(pack2(fast_ex2(e.x), fast_ex2(e.y)), S[i], mul2(x2, B[i]));
+            s = fma2(S[i], C[i], s);
+          }
+          const float2 r = unpack2(s);
+          acc[j] = r.x + r.y;
+        }
+        // four sums over four lanes, one left on each lane: lane l ends with token t4 + l
+        const float x0 = (lane4 & 1) ? acc[0] : acc[1], x1 = (lane4 & 1) ? acc[2] : acc[3];
+        const float g0 = __shfl_xor_sync(0xffffffffu, x0, 1), g1 = __shfl_xor_sync(0xffffffffu, x1, 1);
+        const float h0 = ((lane4 & 1) ? acc[1] : acc[0]) + g0, h1 = ((lane4 & 1) ? acc[3] : acc[2]) + g1;
+        const float g2 = __shfl_xor_sync(0xffffffffu, (lane4 & 2) ? h0 : h1, 2);
+        const float y = ((lane4 & 2) ? h1 : h0) + g2;
+        float2* uz = &sm.uz[b][t4 + lane4][ch];
+        const float2 v = *uz;
+        uz->x = fmaf(D, v.x, y) * v.y;
       }
     }
+    tile_barrier<8 * CH>();     // the last tile is finished
 #pragma unroll
-    for (int k = 0; k < NBC; ++k) {
-      const int idx = tid + k * NT;
-      const int tt = idx / (8 * NS), w = idx - tt * 8 * NS, half = w / (4 * NS), n = w - half * 4 * NS;
-      rbc[k] = idx < SC_TT * 8 * NS && t0 + tt < p.rows && n < N ? load_source1<T>(a.bc, p.row0 + t0 + tt, half * N + n) : 0.f;
+    for (int i = 0; i < NP; ++i) {
+      const float2 v = unpack2(S[i]);
+      if (live && lane4 * NS + 2 * i < N) sp[2 * i] = v.x;
+      if (live && lane4 * NS + 2 * i + 1 < N) sp[2 * i + 1] = v.y;
+    }
+    return;
+  }
+  // ---------------- feed
+  const int tid = threadIdx.x - NT;
+  constexpr int STEP = NT / Q;
+  const int lt = tid / Q, lq = (tid % Q) * 4, lc = c0 + lq;   // tokens lt + r * STEP, channels lc .. lc + 3
+  float bias[4];
+#pragma unroll
+  for (int e = 0; e < 4; ++e) bias[e] = lc + e < a.inner ? a.dt_bias[lc + e] : 0.f;
+  const T* ug = reinterpret_cast<const T*>(a.u);
+  T* yg = reinterpret_cast<T*>(a.y);
+  const bool vec_y = FAST || (a.inner % 4 == 0 && a.ldy % 4 == 0 && (reinterpret_cast<uintptr_t>(a.y) & 15) == 0);
+  constexpr int NBC = (SC_TT * 2 * NS + NT - 1) / NT;   // B / C groups of four that a thread loads
+  Raw<T, 4> ru[FAST ? ROWS : 1], rd[FAST ? ROWS : 1], rz[FAST ? ROWS : 1], rbc[FAST ? NBC : 1];
+  auto fetch = [&](int t0) {   // rows beyond the portion: its last one again
+    if constexpr (FAST) {
+      const int cc = min(lc, a.inner - 4);
+#pragma unroll
+      for (int r = 0; r < ROWS; ++r) {
+        const long long row = p.row0 + min(t0 + lt + r * STEP, p.rows - 1);
+        ru[r].load(ug + row * a.ldu + cc);
+        rd[r].load(reinterpret_cast<const T*>(a.dt.p) + row * a.dt.ld + cc);
+        rz[r].load(reinterpret_cast<const T*>(a.z.p) + row * a.z.ld + cc);
+      }
+#pragma unroll
+      for (int k = 0; k < NBC; ++k) {
+        const int idx = min(tid + k * NT, SC_TT * 2 * NS - 1);
+        const int tt = idx / (2 * NS), w = idx - tt * 2 * NS;
+        rbc[k].load(reinterpret_cast<const T*>(a.bc.p) + (p.row0 + min(t0 + tt, p.rows - 1)) * a.bc.ld + 4 * w);
+      }
     }
   };
   auto put = [&](int t0, int b) {
-    const bool in = t0 + lt < p.rows;
 #pragma unroll
-    for (int e = 0; e < 4; ++e) {
-      const float dt = in ? softplus_f32(rd[e] + bias[e]) : 0.f;   // tokens beyond the portion leave the state alone
-      du_s[b][lt][lq + e] = make_float2(dt, dt * ru[e]);
-      u_s[b][lt][lq + e] = ru[e];
-      z_s[b][lt][lq + e] = silu_f32(rz[e]);
+    for (int r = 0; r < ROWS; ++r) {
+      const int t = lt + r * STEP;
+      const bool in = t0 + t < p.rows;
+      float u4[4], d4[4], z4[4];
+      if constexpr (FAST) {
+        ru[r].get(u4); rd[r].get(d4); rz[r].get(z4);
+      } else {
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const bool have = in && lc + e < a.inner;
+          const long long row = p.row0 + t0 + t;
+          u4[e] = have ? Elem<T>::get(ug + row * a.ldu + lc + e) : 0.f;
+          d4[e] = have ? load_source1<T>(a.dt, row, lc + e) : 0.f;
+          z4[e] = have ? load_source1<T>(a.z, row, lc + e) : 0.f;
+        }
+      }
+#pragma unroll
+      for (int e = 0; e < 4; e += 2) {
+        // tokens beyond the portion leave the state alone (dt = 0)
+        const float d0 = in ? softplus_f32(d4[e] + bias[e]) : 0.f, d1 = in ? softplus_f32(d4[e + 1] + bias[e + 1]) : 0.f;
+        *reinterpret_cast<float4*>(&sm.du[b][t][lq + e]) = make_float4(d0, d0 * u4[e], d1, d1 * u4[e + 1]);
+        *reinterpret_cast<float4*>(&sm.uz[b][t][lq + e]) = make_float4(u4[e], silu_fast(z4[e]), u4[e + 1], silu_fast(z4[e + 1]));
+      }
     }
+    if constexpr (FAST) {
 #pragma unroll
-    for (int k = 0; k < NBC; ++k) {
-      const int idx = tid + k * NT;
-      if (idx < SC_TT * 8 * NS) (&bc_s[b][0][0][0][0])[idx] = rbc[k];
+      for (int k = 0; k < NBC; ++k) {
+        const int idx = tid + k * NT;
+        float v[4];
+        rbc[k].get(v);
+        if (idx < SC_TT * 2 * NS) *reinterpret_cast<float4*>(&sm.bc[b][0][0][0] + 4 * idx) = make_float4(v[0], v[1], v[2], v[3]);
+      }
+    } else {
+#pragma unroll 1
+      for (int idx = tid; idx < SC_TT * 8 * NS; idx += NT) {
+        const int tt = idx / (8 * NS), w = idx - tt * 8 * NS, half = w / (4 * NS), n = w - half * 4 * NS;
+        (&sm.bc[b][0][0][0])[idx] = t0 + tt < p.rows && n < N ? load_source1<T>(a.bc, p.row0 + t0 + tt, half * N + n) : 0.f;
+      }
     }
   };
-  T* yg = reinterpret_cast<T*>(a.y);
-  const bool vec_y = a.inner % 4 == 0 && a.ldy % 4 == 0 && (reinterpret_cast<uintptr_t>(a.y) & 15) == 0;
-  fetch(0);
-  put(0, 0);
-  __syncthreads();
-  int b = 0;
-  for (int t0 = 0; t0 < p.rows; t0 += SC_TT, b ^= 1) {
-    const bool more = t0 + SC_TT < p.rows;
-    if (more) fetch(t0 + SC_TT);
-#pragma unroll 1
-    for (int t4 = 0; t4 < SC_TT; t4 += 4) {
-      float acc[4];
+  auto flush = [&](int t0, int b) {
 #pragma unroll
-      for (int j = 0; j < 4; ++j) {
-        const float2 du = du_s[b][t4 + j][ch];
-        const float* B = bc_s[b][t4 + j][0][lane4];
-        const float* C = bc_s[b][t4 + j][1][lane4];
-        float s = 0.f;
+    for (int r = 0; r < ROWS; ++r) {
+      const int t = lt + r * STEP;
+      if (t0 + t >= p.rows) continue;
+      T* dst = yg + (long long)(p.row0 + t0 + t) * a.ldy + lc;
+      float o[4];
 #pragma unroll
-        for (int i = 0; i < NS; ++i) {
-          S[i] = fmaf(fast_ex2(du.x * a2[i]), S[i], du.y * B[i]);
-          s = fmaf(S[i], C[i], s);
-        }
-        acc[j] = s;
-      }
-      // four sums over four lanes, one left on each lane: lane l ends with token t4 + l
-      const float x0 = (lane4 & 1) ? acc[0] : acc[1], x1 = (lane4 & 1) ? acc[2] : acc[3];
-      const float g0 = __shfl_xor_sync(0xffffffffu, x0, 1), g1 = __shfl_xor_sync(0xffffffffu, x1, 1);
-      const float h0 = ((lane4 & 1) ? acc[1] : acc[0]) + g0, h1 = ((lane4 & 1) ? acc[3] : acc[2]) + g1;
-      const float g2 = __shfl_xor_sync(0xffffffffu, (lane4 & 2) ? h0 : h1, 2);
-      const float y = ((lane4 & 2) ? h1 : h0) + g2;
-      const int t = t4 + lane4;
-      z_s[b][t][ch] *= fmaf(D, u_s[b][t][ch], y);
-    }
-    if (more) put(t0 + SC_TT, b ^ 1);
-    __syncthreads();
-    if (t0 + lt < p.rows) {
-      T* dst = yg + (long long)(p.row0 + t0 + lt) * a.ldy + lc;
+      for (int e = 0; e < 4; ++e) o[e] = sm.uz[b][t][lq + e].x;
       if (vec_y) {
-        float o[4];
-#pragma unroll
-        for (int e = 0; e < 4; ++e) o[e] = z_s[b][lt][lq + e];
         if (lc < a.inner) Vec<T, 4>::store(dst, o);
       } else {
 #pragma unroll
         for (int e = 0; e < 4; ++e)
-          if (lc + e < a.inner) Elem<T>::put(dst + e, z_s[b][lt][lq + e]);
+          if (lc + e < a.inner) Elem<T>::put(dst + e, o[e]);
       }
     }
+  };
+  fetch(0);
+  put(0, 0);
+  fetch(SC_TT);
+  for (int k = 0; k < n_tiles; ++k) {
+    tile_barrier<8 * CH>();   // the scan takes tile k; tile k - 1 is finished
+    // the buffer of tile k - 1 is read and refilled by the same threads
+    if (k > 0) flush((k - 1) * SC_TT, (k - 1) & 1);
+    if (k + 1 < n_tiles) {
+      put((k + 1) * SC_TT, (k + 1) & 1);
+      fetch((k + 2) * SC_TT);
+    }
   }
-#pragma unroll
-  for (int i = 0; i < NS; ++i)
-    if (live && lane4 * NS + i < N) sp[i] = S[i];
+  tile_barrier<8 * CH>();
+  flush((n_tiles - 1) * SC_TT, (n_tiles - 1) & 1);
 }
 
 // One token per sequence: four lanes a channel, the state read and written once.
@@ -357,7 +525,14 @@ static void launch_conv(const CausalConvArgs& a, cudaStream_t s) {
   const int v = vec && a.taps <= 4 ? 8 : 1;
   const int per = (a.inner + v - 1) / v, threads = std::min(128, (per + 31) / 32 * 32);
   const dim3 grid((per + threads - 1) / threads, a.tiles ? a.n_tiles : a.rows.n);
-  if (v == 8) {
+  if (v == 8 && a.tiles && a.x.k_splits == 0) {
+    switch (a.taps) {
+      case 1: cb::causal_conv_rows_kernel<T, 1><<<grid, threads, 0, s>>>(a); break;
+      case 2: cb::causal_conv_rows_kernel<T, 2><<<grid, threads, 0, s>>>(a); break;
+      case 3: cb::causal_conv_rows_kernel<T, 3><<<grid, threads, 0, s>>>(a); break;
+      default: cb::causal_conv_rows_kernel<T, 4><<<grid, threads, 0, s>>>(a); break;
+    }
+  } else if (v == 8) {
     switch (a.taps) {
       case 1: cb::causal_conv_kernel<T, 8, 1><<<grid, threads, 0, s>>>(a); break;
       case 2: cb::causal_conv_kernel<T, 8, 2><<<grid, threads, 0, s>>>(a); break;
@@ -377,22 +552,44 @@ void causal_conv(const CausalConvArgs& a, cudaStream_t s) {
   a.is_f32 ? launch_conv<float>(a, s) : launch_conv<bf16>(a, s);
 }
 
+template <typename T, int NS, int CH, bool FAST>
+static void launch_scan_ch(const SelectiveScanArgs& a, cudaStream_t s) {
+  constexpr int smem = (int)sizeof(cb::ScanSmem<NS, CH>);
+  static bool granted = false;
+  if (!granted && smem > 48 * 1024) {
+    if (cudaFuncSetAttribute(cb::selective_scan_kernel<T, NS, CH, FAST>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess)
+      throw std::runtime_error("selective_scan: shared memory not available");
+    granted = true;
+  }
+  cb::selective_scan_kernel<T, NS, CH, FAST><<<dim3((a.inner + CH - 1) / CH, a.rows.n), 8 * CH, smem, s>>>(a);
+}
+
 template <typename T, int NS>
 static void launch_scan_ns(const SelectiveScanArgs& a, cudaStream_t s) {
   if (!a.rows.portions) {
     cb::selective_step_kernel<T, NS><<<dim3((a.inner + 63) / 64, a.rows.n), 256, 0, s>>>(a);
-  } else if ((long long)(a.inner + 31) / 32 * a.rows.n >= 148) {
-    cb::selective_scan_kernel<T, NS, 32><<<dim3((a.inner + 31) / 32, a.rows.n), 128, 0, s>>>(a);
-  } else {   // few channels: more, smaller CTAs
-    cb::selective_scan_kernel<T, NS, 8><<<dim3((a.inner + 7) / 8, a.rows.n), 32, 0, s>>>(a);
+    return;
   }
+  auto on = [](const RowSource& r) { return (reinterpret_cast<uintptr_t>(r.p) & 15) == 0 && r.ld % 4 == 0 && r.k_splits == 0; };
+  const bool fast = a.inner % 4 == 0 && a.state == 4 * NS && on(a.dt) && on(a.z) && on(a.bc) && a.ldu % 4 == 0 && a.ldy % 4 == 0 &&
+                    (reinterpret_cast<uintptr_t>(a.u) & 15) == 0 && (reinterpret_cast<uintptr_t>(a.y) & 15) == 0;
+  if constexpr (NS <= 16) {
+    if (fast) {
+      // about two CTAs of 32 channels per SM; fewer channels a CTA while that leaves SMs idle
+      const long long ctas = (long long)((a.inner + 31) / 32) * a.rows.n;
+      if constexpr (sizeof(T) == 2) {
+        if (ctas >= 200) return launch_scan_ch<T, NS, 32, true>(a, s);
+      }
+      return launch_scan_ch<T, NS, 16, true>(a, s);
+    }
+  }
+  launch_scan_ch<T, NS, 16, false>(a, s);
 }
 
 template <typename T>
 static void launch_scan(const SelectiveScanArgs& a, cudaStream_t s) {
   const int per = (a.state + 3) / 4;
-  if (per <= 1) launch_scan_ns<T, 1>(a, s);
-  else if (per <= 2) launch_scan_ns<T, 2>(a, s);
+  if (per <= 2) launch_scan_ns<T, 2>(a, s);
   else if (per <= 4) launch_scan_ns<T, 4>(a, s);
   else if (per <= 6) launch_scan_ns<T, 6>(a, s);
   else if (per <= 8) launch_scan_ns<T, 8>(a, s);

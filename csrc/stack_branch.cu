@@ -11,15 +11,16 @@
 namespace cb {
 
 // One CTA per token row; a row's vectors stay in registers, all loads are issued before the first sum.
-template <typename T, int VEC, int NV>
-__global__ void __launch_bounds__(1024)
+// PART: some source holds split-K partial sums. EMBED: rows start from the embedding.
+template <typename T, int VEC, int NV, bool PART, bool EMBED>
+__global__ void __launch_bounds__(NV == 1 ? 1024 : 512)
 branch_norm_kernel(const cosmos::BranchNormArgs a) {
   __shared__ float2 buf_s[2][32];
   const long long r = blockIdx.x;
   const int tid = threadIdx.x, nt = blockDim.x, d = a.d;
   float* xr = a.x + r * d;
   float v[NV][VEC], b0[NV][VEC], b1[NV][VEC];
-  if (a.embed) {
+  if constexpr (EMBED) {
     long long tok = a.tokens[r];
     if (!index_ok(tok, a.vocab, a.status, SITE_STACK_TOKEN)) tok = 0;
     const T* er = reinterpret_cast<const T*>(a.embed) + tok * a.ld_embed;
@@ -56,11 +57,11 @@ branch_norm_kernel(const cosmos::BranchNormArgs a) {
     for (int i = 0; i < NV; ++i) {
       const int c = (tid + i * nt) * VEC;
       if (c < d) {
-        load_source<T, VEC>(a.normed[0], r, c, b0[i]);
+        load_source<T, VEC, PART>(a.normed[0], r, c, b0[i]);
 #pragma unroll
         for (int e = 0; e < VEC; ++e) s0 = fmaf(b0[i][e], b0[i][e], s0);
         if (a.n_normed > 1) {
-          load_source<T, VEC>(a.normed[1], r, c, b1[i]);
+          load_source<T, VEC, PART>(a.normed[1], r, c, b1[i]);
 #pragma unroll
           for (int e = 0; e < VEC; ++e) s1 = fmaf(b1[i][e], b1[i][e], s1);
         }
@@ -91,11 +92,11 @@ branch_norm_kernel(const cosmos::BranchNormArgs a) {
     if (c < d) {
       if (a.has_plain) {
         float t[VEC];
-        load_source<T, VEC>(a.plain, r, c, t);
+        load_source<T, VEC, PART>(a.plain, r, c, t);
 #pragma unroll
         for (int e = 0; e < VEC; ++e) v[i][e] += t[e];
       }
-      if (a.embed || a.n_normed || a.has_plain) Vec<float, VEC>::store(xr + c, v[i]);
+      if (EMBED || a.n_normed || a.has_plain) Vec<float, VEC>::store(xr + c, v[i]);
 #pragma unroll
       for (int e = 0; e < VEC; ++e) ss = fmaf(v[i][e], v[i][e], ss);
     }
@@ -120,8 +121,8 @@ branch_norm_kernel(const cosmos::BranchNormArgs a) {
 }
 
 // One CTA per token row: the whole q row and the whole k row.
-template <typename T, int VEC, int NV>
-__global__ void __launch_bounds__(1024)
+template <typename T, int VEC, int NV, bool PART>
+__global__ void __launch_bounds__(NV == 1 ? 1024 : 512)
 qk_norm_post_kernel(const cosmos::QkNormArgs a) {
   __shared__ float2 buf_s[32];
   const long long r = blockIdx.x;
@@ -133,12 +134,12 @@ qk_norm_post_kernel(const cosmos::QkNormArgs a) {
   for (int i = 0; i < NV; ++i) {
     const int c = (tid + i * nt) * VEC;
     if (c < qc) {
-      load_source<T, VEC>(a.q, r, c, q[i]);
+      load_source<T, VEC, PART>(a.q, r, c, q[i]);
 #pragma unroll
       for (int e = 0; e < VEC; ++e) sq = fmaf(q[i][e], q[i][e], sq);
     }
     if (c < kc) {
-      load_source<T, VEC>(a.k, r, c, k[i]);
+      load_source<T, VEC, PART>(a.k, r, c, k[i]);
 #pragma unroll
       for (int e = 0; e < VEC; ++e) sk = fmaf(k[i][e], k[i][e], sk);
     }
@@ -147,13 +148,13 @@ qk_norm_post_kernel(const cosmos::QkNormArgs a) {
   float rq = 1.f / sqrtf(ss.x / (float)qc + a.eps);
   const float rk = 1.f / sqrtf(ss.y / (float)kc + a.eps);
   if (a.temp_every > 0) {
-    const long long step = (a.positions[r] + 1) / a.temp_every;
+    const unsigned step = (unsigned)(a.positions[r] + 1) / (unsigned)a.temp_every;   // positions fit 32 bits
     rq *= 1.f + a.temp_coef * logf((float)(step + 1));
   }
   const long long slot = a.slots[r];
   const bool ok = index_ok(slot, a.n_slots, a.status, SITE_STACK_SLOT);
-  const long long page = ok ? slot / a.page_size : 0;
-  const int off = ok ? (int)(slot - page * a.page_size) : 0;
+  const unsigned page = ok ? (unsigned)slot / (unsigned)a.page_size : 0u;
+  const int off = ok ? (int)((unsigned)slot - page * (unsigned)a.page_size) : 0;
   T* qo = reinterpret_cast<T*>(a.q_out) + r * qc;
 #pragma unroll
   for (int i = 0; i < NV; ++i) {
@@ -167,7 +168,7 @@ qk_norm_post_kernel(const cosmos::QkNormArgs a) {
     }
     if (c < kc && ok) {
       const int g = c / a.dim;
-      const long long row = ((page * a.G + g) * a.page_size + off) * (long long)a.dim + (c - g * a.dim);
+      const long long row = (((long long)page * a.G + g) * a.page_size + off) * (long long)a.dim + (c - g * a.dim);
       Vec<T, VEC>::store(reinterpret_cast<T*>(a.v_cache) + row, k[i]);
       Vec<float, VEC>::load(a.wk + c, w);
 #pragma unroll
@@ -190,50 +191,61 @@ static int row_threads(int cols, int vec, int nv) {
   return std::max(32, ((cols + per - 1) / per + 31) / 32 * 32);
 }
 
-template <typename T>
+template <typename T, bool PART, bool EMBED>
 static void launch_branch(const BranchNormArgs& a, cudaStream_t s) {
   bool vec = a.d % 8 == 0 && a.ldh % 8 == 0 && a.ld_embed % 8 == 0 && on(a.x, 16) && on(a.embed, 16);
   for (int i = 0; i < 2; ++i) vec = vec && on(a.gamma[i], 16) && on(a.h[i], 16) && on(a.normed_w[i], 16) && vec8_source(a.normed[i]);
   if (a.has_plain) vec = vec && vec8_source(a.plain);
   const unsigned rows = (unsigned)a.rows;
-  if (vec && a.d <= 8192 && a.rows <= 296)
-    cb::branch_norm_kernel<T, 8, 1><<<rows, row_threads(a.d, 8, 1), 0, s>>>(a);
-  else if (vec && a.d <= 16384)
-    cb::branch_norm_kernel<T, 8, 2><<<rows, row_threads(a.d, 8, 2), 0, s>>>(a);
+  if (vec && a.d <= 8192 && (a.rows <= 296 || a.d <= 1024))
+    cb::branch_norm_kernel<T, 8, 1, PART, EMBED><<<rows, row_threads(a.d, 8, 1), 0, s>>>(a);
+  else if (vec && a.d <= 8192)
+    cb::branch_norm_kernel<T, 8, 2, PART, EMBED><<<rows, row_threads(a.d, 8, 2), 0, s>>>(a);
   else if (a.d <= 1024)
-    cb::branch_norm_kernel<T, 1, 1><<<rows, row_threads(a.d, 1, 1), 0, s>>>(a);
+    cb::branch_norm_kernel<T, 1, 1, PART, EMBED><<<rows, row_threads(a.d, 1, 1), 0, s>>>(a);
   else if (a.d <= 16384)
-    cb::branch_norm_kernel<T, 1, 16><<<rows, row_threads(a.d, 1, 16), 0, s>>>(a);
+    cb::branch_norm_kernel<T, 1, 32, PART, EMBED><<<rows, row_threads(a.d, 1, 32), 0, s>>>(a);
   else
     throw std::runtime_error("branch_norm: rows of up to 16384 columns");
 }
 
 void branch_norm(const BranchNormArgs& a, cudaStream_t s) {
   if (a.rows <= 0) return;
-  a.is_f32 ? launch_branch<float>(a, s) : launch_branch<bf16>(a, s);
+  bool part = a.has_plain && a.plain.k_splits > 0;
+  for (int i = 0; i < a.n_normed; ++i) part = part || a.normed[i].k_splits > 0;
+  if (a.embed) {
+    if (a.n_normed || a.has_plain) throw std::runtime_error("branch_norm: the embedding starts a row");
+    a.is_f32 ? launch_branch<float, false, true>(a, s) : launch_branch<bf16, false, true>(a, s);
+  } else if (part) {
+    a.is_f32 ? launch_branch<float, true, false>(a, s) : launch_branch<bf16, true, false>(a, s);
+  } else {
+    a.is_f32 ? launch_branch<float, false, false>(a, s) : launch_branch<bf16, false, false>(a, s);
+  }
 }
 
-template <typename T>
+template <typename T, bool PART>
 static void launch_qk(const QkNormArgs& a, cudaStream_t s) {
   const int cols = std::max(a.H, a.G) * a.dim;
   const bool vec = a.dim % 8 == 0 && vec8_source(a.q) && vec8_source(a.k) && on(a.wq, 16) && on(a.wk, 16) && on(a.q_out, 16) &&
                    on(a.k_cache, 16) && on(a.v_cache, 16);
   const unsigned rows = (unsigned)a.n;
-  if (vec && cols <= 8192 && a.n <= 296)
-    cb::qk_norm_post_kernel<T, 8, 1><<<rows, row_threads(cols, 8, 1), 0, s>>>(a);
-  else if (vec && cols <= 16384)
-    cb::qk_norm_post_kernel<T, 8, 2><<<rows, row_threads(cols, 8, 2), 0, s>>>(a);
+  if (vec && cols <= 8192)
+    cb::qk_norm_post_kernel<T, 8, 1, PART><<<rows, row_threads(cols, 8, 1), 0, s>>>(a);
   else if (cols <= 1024)
-    cb::qk_norm_post_kernel<T, 1, 1><<<rows, row_threads(cols, 1, 1), 0, s>>>(a);
+    cb::qk_norm_post_kernel<T, 1, 1, PART><<<rows, row_threads(cols, 1, 1), 0, s>>>(a);
   else if (cols <= 16384)
-    cb::qk_norm_post_kernel<T, 1, 16><<<rows, row_threads(cols, 1, 16), 0, s>>>(a);
+    cb::qk_norm_post_kernel<T, 1, 32, PART><<<rows, row_threads(cols, 1, 32), 0, s>>>(a);
   else
     throw std::runtime_error("qk_norm_post: projections of up to 16384 columns");
 }
 
 void qk_norm_post(const QkNormArgs& a, cudaStream_t s) {
   if (a.n <= 0) return;
-  a.is_f32 ? launch_qk<float>(a, s) : launch_qk<bf16>(a, s);
+  if (a.n_slots > 0xffffffffll || a.temp_every > 0x7fffffff) throw std::runtime_error("qk_norm_post: too many cache slots");
+  if (a.q.k_splits || a.k.k_splits)
+    a.is_f32 ? launch_qk<float, true>(a, s) : launch_qk<bf16, true>(a, s);
+  else
+    a.is_f32 ? launch_qk<float, false>(a, s) : launch_qk<bf16, false>(a, s);
 }
 
 }  // namespace cosmos

@@ -69,6 +69,34 @@ template <> struct Vec<bf16, 8> {
   }
 };
 
+// Values still in their storage form: a load whose conversion comes later does not hold up the loads behind it.
+template <typename T, int VEC> struct Raw;
+template <> struct Raw<bf16, 4> {
+  uint2 v;
+  __device__ __forceinline__ void load(const bf16* p) { v = *reinterpret_cast<const uint2*>(p); }
+  __device__ __forceinline__ void get(float (&o)[4]) const { o[0] = bf16lo(v.x); o[1] = bf16hi(v.x); o[2] = bf16lo(v.y); o[3] = bf16hi(v.y); }
+};
+template <> struct Raw<float, 4> {
+  float4 v;
+  __device__ __forceinline__ void load(const float* p) { v = *reinterpret_cast<const float4*>(p); }
+  __device__ __forceinline__ void get(float (&o)[4]) const { o[0] = v.x; o[1] = v.y; o[2] = v.z; o[3] = v.w; }
+};
+template <> struct Raw<bf16, 8> {
+  uint4 v;
+  __device__ __forceinline__ void load(const bf16* p) { v = *reinterpret_cast<const uint4*>(p); }
+  __device__ __forceinline__ void get(float (&o)[8]) const {
+    o[0] = bf16lo(v.x); o[1] = bf16hi(v.x); o[2] = bf16lo(v.y); o[3] = bf16hi(v.y);
+    o[4] = bf16lo(v.z); o[5] = bf16hi(v.z); o[6] = bf16lo(v.w); o[7] = bf16hi(v.w);
+  }
+};
+template <> struct Raw<float, 8> {
+  float4 a, b;
+  __device__ __forceinline__ void load(const float* p) { a = reinterpret_cast<const float4*>(p)[0]; b = reinterpret_cast<const float4*>(p)[1]; }
+  __device__ __forceinline__ void get(float (&o)[8]) const {
+    o[0] = a.x; o[1] = a.y; o[2] = a.z; o[3] = a.w; o[4] = b.x; o[5] = b.y; o[6] = b.z; o[7] = b.w;
+  }
+};
+
 __device__ __forceinline__ float warp_add(float v) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
@@ -84,9 +112,10 @@ __device__ __forceinline__ float silu_f32(float z) { return z / (1.f + expf(-z))
 __device__ __forceinline__ float sigmoid_f32(float z) { return 1.f / (1.f + expf(-z)); }
 
 // VEC consecutive values of a RowSource (stack.h): the row itself, or the sum of its split-K parts.
-template <typename T, int VEC>
+// PART false: known to be finished values.
+template <typename T, int VEC, bool PART = true>
 __device__ __forceinline__ void load_source(const cosmos::RowSource& s, long long row, int col, float (&v)[VEC]) {
-  if (s.k_splits == 0) {
+  if (!PART || s.k_splits == 0) {
     Vec<T, VEC>::load(reinterpret_cast<const T*>(s.p) + row * s.ld + col, v);
     return;
   }
