@@ -366,15 +366,15 @@ def memory_slices(vdim: int) -> int:
 
 
 def matrix_memory(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, gates: torch.Tensor, gate_bias: torch.Tensor, cap: float,
-                  state: torch.Tensor, norm: torch.Tensor, peak: torch.Tensor, rows: StepRows, n: int, dtype) -> torch.Tensor:
+                  state: torch.Tensor, norm: torch.Tensor, peak: torch.Tensor, rows: StepRows, n: int, dtype, impl: int = 0) -> torch.Tensor:
     """mLSTM over rows q, k [n, >= H dim], v [n, >= H vdim] (or partial sums) and fp32 gate rows [n, >= 2 H] (input gates, then
     forget gates): log gates i = cap tanh(. / cap), f = logsigmoid(cap tanh(. / cap)), running maximum m = max(f + m, i) from 0,
     S = exp(f + m' - m) S + exp(i - m) k v^T, n likewise, o = S^T q / (max(|n . q|, exp(-m)) + 1e-6), q over sqrt(dim).
-    state [slots, H, dim, vdim], norm [slots, H, slices, dim], peak [slots, H, slices] fp32. Returns [n, H * vdim]."""
+    state [slots, H, dim, vdim], norm [slots, H, slices, dim], peak [slots, H, slices] fp32. Returns [n, H * vdim]. impl 1 forces the CUDA-core kernel."""
     heads, dim, vdim = state.shape[1:]
     if _cuda(q):
         return _k().matrix_memory(q, k, v, gates, gate_bias, dim ** -0.5, float(cap), state, norm, peak, rows.state_slots, rows.portions,
-                                  rows.lens, n, dtype == torch.float32)
+                                  rows.lens, n, dtype == torch.float32, impl)
     qr = _rows(q)[:, :heads * dim].reshape(n, heads, dim) * dim ** -0.5
     kr, vr = _rows(k)[:, :heads * dim].reshape(n, heads, dim), _rows(v)[:, :heads * vdim].reshape(n, heads, vdim)
     g = cap * torch.tanh((_rows(gates)[:, :2 * heads] + gate_bias) / cap)

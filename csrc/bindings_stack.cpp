@@ -460,10 +460,10 @@ void selective_scan(const Tensor& u, const Tensor& dt, const Tensor& z, const Te
 }
 
 // See MatrixMemoryArgs -> o [n, H * vdim] (row stride padded to 8). S [slots, H, dim, vdim], nrm [slots, H, slices, dim],
-// m [slots, H, slices] fp32.
+// m [slots, H, slices] fp32. impl 0 = tcgen05 where it applies, 1 = CUDA cores.
 Tensor matrix_memory(const Tensor& q, const Tensor& k, const Tensor& v, const Tensor& gates, const Tensor& gate_bias, double q_scale,
                      double cap, Tensor S, Tensor nrm, Tensor m, const Tensor& state_slots, const OptT& portions, const OptT& lens,
-                     int64_t n, bool f32) {
+                     int64_t n, bool f32, int64_t impl) {
   c10::cuda::CUDAGuard guard(q.device());
   cosmos::MatrixMemoryArgs a;
   TORCH_CHECK(S.dim() == 4 && S.scalar_type() == at::kFloat && S.is_contiguous(), "S must be fp32 [slots, H, dim, vdim]");
@@ -484,7 +484,12 @@ Tensor matrix_memory(const Tensor& q, const Tensor& k, const Tensor& v, const Te
   Tensor o = padded_rows(n, (int64_t)a.H * a.vdim, S.options().dtype(f32 ? at::kFloat : at::kBFloat16));
   a.o = o.data_ptr(); a.ldo = o.stride(0);
   a.status = status_ptr(q);
-  cosmos::matrix_memory(a, cur_stream());
+  a.n_rows = n;
+  // the chunked kernel once portions fill a good part of a chunk
+  if (impl == 0 && n >= 48 * (int64_t)a.rows.n && cosmos::matrix_memory_tc_supported(a))
+    cosmos::matrix_memory_tc(a, cur_stream());
+  else
+    cosmos::matrix_memory(a, cur_stream());
   return o;
 }
 

@@ -253,15 +253,18 @@ struct MatrixMemoryArgs {
   float* S = nullptr;
   float* n = nullptr;
   float* m = nullptr;
-  void* o = nullptr;                   // [rows, H * vdim]
-  long long ldo = 0;
+  void* o = nullptr;                   // [n_rows, H * vdim]
+  long long ldo = 0, n_rows = 0;
   StepRows rows;
   bool is_f32 = false;
   int* status = nullptr;
 };
 constexpr int MEMORY_SLICE = 32;
 constexpr int MEMORY_MAX_DIM = 512;
-void matrix_memory(const MatrixMemoryArgs& a, cudaStream_t s);
+void matrix_memory(const MatrixMemoryArgs& a, cudaStream_t s);      // CUDA cores: any sizes, bf16 or fp32, portions and decode steps
+// tcgen05, chunks of 128 tokens (matrix_memory_tc.cu): bf16 portions, dim 64 / 128 / 256, vdim a multiple of MEMORY_SLICE.
+bool matrix_memory_tc_supported(const MatrixMemoryArgs& a);
+void matrix_memory_tc(const MatrixMemoryArgs& a, cudaStream_t s);
 
 // y = o / rms(o of the head) * w * sigmoid(g)
 struct HeadNormGateArgs {
