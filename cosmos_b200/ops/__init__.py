@@ -143,7 +143,7 @@ STATUS_MESSAGES = {
 STATUS_SITES = {1: "kv_cache_write slot", 2: "decode_qkv_post slot", 3: "paged_decode page id",
                 4: "paged_decode (tensor-core) page id", 5: "decoder stack token id", 6: "decoder stack cache slot",
                 7: "windowed attention page id", 8: "expert id of a routing table", 9: "expert-sorted row",
-                15: "self-test"}
+                10: "decoder stack state slot", 15: "self-test"}
 
 
 def check_status(reset: bool = True) -> None:

@@ -297,34 +297,43 @@ selective_scan_kernel(const cosmos::SelectiveScanArgs a) {
     for (int k = 0; k < n_tiles; ++k) {
       const int b = k & 1;
       tile_barrier<8 * CH>();   // tile k is in place
-#pragma unroll 1
+      // the next four tokens' rows are read before the current four are finished (the store of an output would hold them up)
+      float2 du[4];
+      uint64_t B[4][NP], C[4][NP];
+      auto rows = [&](int t4) {
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          du[j] = sm.du[b][t4 + j][ch];
+          load_pairs<NP>(&sm.bc[b][t4 + j][0][lane4 * NS], B[j]);
+          load_pairs<NP>(&sm.bc[b][t4 + j][1][lane4 * NS], C[j]);
+        }
+      };
+      rows(0);
+#pragma unroll 2
       for (int t4 = 0; t4 < SC_TT; t4 += 4) {
+        float2* uz = &sm.uz[b][t4 + lane4][ch];
+        const float2 v = *uz;
         float acc[4];
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
-          const float2 du = sm.du[b][t4 + j][ch];
-          uint64_t B[NP], C[NP];
-          load_pairs<NP>(&sm.bc[b][t4 + j][0][lane4 * NS], B);
-          load_pairs<NP>(&sm.bc[b][t4 + j][1][lane4 * NS], C);
-          const uint64_t dt2 = pack2(du.x, du.x), x2 = pack2(du.y, du.y);
+          const uint64_t dt2 = pack2(du[j].x, du[j].x), x2 = pack2(du[j].y, du[j].y);
           uint64_t s = 0ull;
 #pragma unroll
           for (int i = 0; i < NP; ++i) {
             const float2 e = unpack2(mul2(dt2, a2[i]));
-            S[i] = fma2(pack2(fast_ex2(e.x), fast_ex2(e.y)), S[i], mul2(x2, B[i]));
-            s = fma2(S[i], C[i], s);
+            S[i] = fma2(pack2(fast_ex2(e.x), fast_ex2(e.y)), S[i], mul2(x2, B[j][i]));
+            s = fma2(S[i], C[j][i], s);
           }
           const float2 r = unpack2(s);
           acc[j] = r.x + r.y;
         }
+        rows(min(t4 + 4, SC_TT - 4));
         // four sums over four lanes, one left on each lane: lane l ends with token t4 + l
         const float x0 = (lane4 & 1) ? acc[0] : acc[1], x1 = (lane4 & 1) ? acc[2] : acc[3];
         const float g0 = __shfl_xor_sync(0xffffffffu, x0, 1), g1 = __shfl_xor_sync(0xffffffffu, x1, 1);
         const float h0 = ((lane4 & 1) ? acc[1] : acc[0]) + g0, h1 = ((lane4 & 1) ? acc[3] : acc[2]) + g1;
         const float g2 = __shfl_xor_sync(0xffffffffu, (lane4 & 2) ? h0 : h1, 2);
         const float y = ((lane4 & 2) ? h1 : h0) + g2;
-        float2* uz = &sm.uz[b][t4 + lane4][ch];
-        const float2 v = *uz;
         uz->x = fmaf(D, v.x, y) * v.y;
       }
     }
