@@ -236,7 +236,7 @@ __device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
   return r;
 }
 
-// NP pairs from shared memory
+// NP pairs in storage form from shared memory (8-byte aligned) as fp32 pairs.
 template <int NP>
 __device__ __forceinline__ void load_pairs(const float* p, uint64_t (&v)[NP]) {
   if constexpr (NP % 2 == 0) {
@@ -250,6 +250,25 @@ __device__ __forceinline__ void load_pairs(const float* p, uint64_t (&v)[NP]) {
     for (int i = 0; i < NP; ++i) v[i] = *reinterpret_cast<const unsigned long long*>(p + 2 * i);
   }
 }
+template <int NP>
+__device__ __forceinline__ void load_pairs(const bf16* p, uint64_t (&v)[NP]) {
+  uint32_t w[NP];
+  if constexpr (NP % 4 == 0) {
+#pragma unroll
+    for (int i = 0; i < NP; i += 4) {
+      const uint4 x = *reinterpret_cast<const uint4*>(p + 2 * i);
+      w[i] = x.x; w[i + 1] = x.y; w[i + 2] = x.z; w[i + 3] = x.w;
+    }
+  } else {
+#pragma unroll
+    for (int i = 0; i < NP; i += 2) {
+      const uint2 x = *reinterpret_cast<const uint2*>(p + 2 * i);
+      w[i] = x.x; w[i + 1] = x.y;
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < NP; ++i) v[i] = pack2(bf16lo(w[i]), bf16hi(w[i]));
+}
 
 constexpr int SC_TT = 32;   // tokens per tile
 
@@ -259,11 +278,13 @@ __device__ __forceinline__ void tile_barrier() {
   asm volatile("barrier.sync 1, %0;" ::"n"(N) : "memory");
 }
 
-template <int NS, int CH>
+// Row strides are such that the four lanes of a channel, which finish four different tokens, meet different banks.
+template <typename T, int NS, int CH>
 struct ScanSmem {
-  float2 du[2][SC_TT][CH];            // dt, dt * u
-  float2 uz[2][SC_TT][CH];            // u, silu(z); then the finished output in .x
-  float bc[2][SC_TT][2][4 * NS];      // B | C, NS values per lane
+  float2 du[2][SC_TT][CH];                   // dt, dt * u
+  float2 uz[2][SC_TT][CH + 4];               // u, silu(z)
+  float y[2][SC_TT][CH + 8];                 // finished output
+  __align__(16) T bc[2][SC_TT][4][2 * NS];   // NS values of B, then of C, for each of a channel's four lanes
 };
 
 // FAST: finished, aligned rows and N = 4 NS, loaded a tile ahead; otherwise rows are loaded when their tile is made.
@@ -273,7 +294,8 @@ selective_scan_kernel(const cosmos::SelectiveScanArgs a) {
   constexpr int NT = 4 * CH, NP = NS / 2, Q = CH / 4, ROWS = SC_TT * Q / NT;   // threads of a half; a feeder loads ROWS x 4 values
   static_assert(NS % 2 == 0 && NT % 32 == 0 && ROWS * NT == SC_TT * Q, "tile shape");
   extern __shared__ __align__(16) uint8_t sm_raw[];
-  ScanSmem<NS, CH>& sm = *reinterpret_cast<ScanSmem<NS, CH>*>(sm_raw);
+  using Smem = ScanSmem<T, NS, CH>;
+  Smem& sm = *reinterpret_cast<Smem*>(sm_raw);
   const Portion p = get_portion(a.rows, blockIdx.y);
   if (p.rows <= 0) return;
   const long long slot = get_state_slot(a.rows, p.seq, a.status);
@@ -297,22 +319,20 @@ selective_scan_kernel(const cosmos::SelectiveScanArgs a) {
     for (int k = 0; k < n_tiles; ++k) {
       const int b = k & 1;
       tile_barrier<8 * CH>();   // tile k is in place
-      // the next four tokens' rows are read before the current four are finished (the store of an output would hold them up)
+      // the next four tokens' rows are read before the current four's output is stored
       float2 du[4];
-      uint64_t B[4][NP], C[4][NP];
+      uint64_t BC[4][2 * NP];
       auto rows = [&](int t4) {
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
           du[j] = sm.du[b][t4 + j][ch];
-          load_pairs<NP>(&sm.bc[b][t4 + j][0][lane4 * NS], B[j]);
-          load_pairs<NP>(&sm.bc[b][t4 + j][1][lane4 * NS], C[j]);
+          load_pairs<2 * NP>(&sm.bc[b][t4 + j][lane4][0], BC[j]);
         }
       };
       rows(0);
 #pragma unroll 2
       for (int t4 = 0; t4 < SC_TT; t4 += 4) {
-        float2* uz = &sm.uz[b][t4 + lane4][ch];
-        const float2 v = *uz;
+        const float2 v = sm.uz[b][t4 + lane4][ch];
         float acc[4];
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
@@ -321,8 +341,8 @@ selective_scan_kernel(const cosmos::SelectiveScanArgs a) {
 #pragma unroll
           for (int i = 0; i < NP; ++i) {
             const float2 e = unpack2(mul2(dt2, a2[i]));
-            S[i] = fma2(pack2(fast_ex2(e.x), fast_ex2(e.y)), S[i], mul2(x2, B[j][i]));
-            s = fma2(S[i], C[j][i], s);
+            S[i] = fma2(pack2(fast_ex2(e.x), fast_ex2(e.y)), S[i], mul2(x2, BC[j][i]));
+            s = fma2(S[i], BC[j][NP + i], s);
           }
           const float2 r = unpack2(s);
           acc[j] = r.x + r.y;
@@ -334,7 +354,7 @@ selective_scan_kernel(const cosmos::SelectiveScanArgs a) {
         const float h0 = ((lane4 & 1) ? acc[1] : acc[0]) + g0, h1 = ((lane4 & 1) ? acc[3] : acc[2]) + g1;
         const float g2 = __shfl_xor_sync(0xffffffffu, (lane4 & 2) ? h0 : h1, 2);
         const float y = ((lane4 & 2) ? h1 : h0) + g2;
-        uz->x = fmaf(D, v.x, y) * v.y;
+        sm.y[b][t4 + lane4][ch] = fmaf(D, v.x, y) * v.y;
       }
     }
     tile_barrier<8 * CH>();     // the last tile is finished
@@ -394,27 +414,44 @@ selective_scan_kernel(const cosmos::SelectiveScanArgs a) {
           z4[e] = have ? load_source1<T>(a.z, row, lc + e) : 0.f;
         }
       }
+      float d[4], z[4];
 #pragma unroll
-      for (int e = 0; e < 4; e += 2) {
-        // tokens beyond the portion leave the state alone (dt = 0)
-        const float d0 = in ? softplus_f32(d4[e] + bias[e]) : 0.f, d1 = in ? softplus_f32(d4[e + 1] + bias[e + 1]) : 0.f;
-        *reinterpret_cast<float4*>(&sm.du[b][t][lq + e]) = make_float4(d0, d0 * u4[e], d1, d1 * u4[e + 1]);
-        *reinterpret_cast<float4*>(&sm.uz[b][t][lq + e]) = make_float4(u4[e], silu_fast(z4[e]), u4[e + 1], silu_fast(z4[e + 1]));
+      for (int e = 0; e < 4; ++e) {
+        d[e] = in ? softplus_f32(d4[e] + bias[e]) : 0.f;   // tokens beyond the portion leave the state alone (dt = 0)
+        z[e] = silu_fast(z4[e]);
+      }
+      // pieces of two channels; every second group of four threads starts with its upper piece, so that eight threads' 16-byte
+      // stores meet all banks
+      const bool up = (tid >> 2) & 1;
+#pragma unroll
+      for (int k = 0; k < 2; ++k) {
+        const int e = (k == 0) == up ? 2 : 0;
+        const float da = e ? d[2] : d[0], db = e ? d[3] : d[1], ua = e ? u4[2] : u4[0], ub = e ? u4[3] : u4[1];
+        *reinterpret_cast<float4*>(&sm.du[b][t][lq + e]) = make_float4(da, da * ua, db, db * ub);
+        *reinterpret_cast<float4*>(&sm.uz[b][t][lq + e]) = make_float4(ua, e ? z[2] : z[0], ub, e ? z[3] : z[1]);
       }
     }
     if constexpr (FAST) {
 #pragma unroll
       for (int k = 0; k < NBC; ++k) {
         const int idx = tid + k * NT;
+        if (idx >= SC_TT * 2 * NS) break;
+        const int tt = idx / (2 * NS), w = idx - tt * 2 * NS, half = w / NS, n = (w - half * NS) * 4;
         float v[4];
         rbc[k].get(v);
-        if (idx < SC_TT * 2 * NS) *reinterpret_cast<float4*>(&sm.bc[b][0][0][0] + 4 * idx) = make_float4(v[0], v[1], v[2], v[3]);
+#pragma unroll
+        for (int e = 0; e < 4; e += 2) {
+          T* dst = &sm.bc[b][tt][(n + e) / NS][half * NS + (n + e) % NS];
+          Elem<T>::put(dst, v[e]);
+          Elem<T>::put(dst + 1, v[e + 1]);
+        }
       }
     } else {
 #pragma unroll 1
       for (int idx = tid; idx < SC_TT * 8 * NS; idx += NT) {
         const int tt = idx / (8 * NS), w = idx - tt * 8 * NS, half = w / (4 * NS), n = w - half * 4 * NS;
-        (&sm.bc[b][0][0][0])[idx] = t0 + tt < p.rows && n < N ? load_source1<T>(a.bc, p.row0 + t0 + tt, half * N + n) : 0.f;
+        Elem<T>::put(&sm.bc[b][tt][n / NS][half * NS + n % NS],
+                     t0 + tt < p.rows && n < N ? load_source1<T>(a.bc, p.row0 + t0 + tt, half * N + n) : 0.f);
       }
     }
   };
@@ -425,8 +462,7 @@ selective_scan_kernel(const cosmos::SelectiveScanArgs a) {
       if (t0 + t >= p.rows) continue;
       T* dst = yg + (long long)(p.row0 + t0 + t) * a.ldy + lc;
       float o[4];
-#pragma unroll
-      for (int e = 0; e < 4; ++e) o[e] = sm.uz[b][t][lq + e].x;
+      Vec<float, 4>::load(&sm.y[b][t][lq], o);
       if (vec_y) {
         if (lc < a.inner) Vec<T, 4>::store(dst, o);
       } else {
@@ -441,7 +477,6 @@ selective_scan_kernel(const cosmos::SelectiveScanArgs a) {
   fetch(SC_TT);
   for (int k = 0; k < n_tiles; ++k) {
     tile_barrier<8 * CH>();   // the scan takes tile k; tile k - 1 is finished
-    // the buffer of tile k - 1 is read and refilled by the same threads
     if (k > 0) flush((k - 1) * SC_TT, (k - 1) & 1);
     if (k + 1 < n_tiles) {
       put((k + 1) * SC_TT, (k + 1) & 1);
@@ -563,7 +598,7 @@ void causal_conv(const CausalConvArgs& a, cudaStream_t s) {
 
 template <typename T, int NS, int CH, bool FAST>
 static void launch_scan_ch(const SelectiveScanArgs& a, cudaStream_t s) {
-  constexpr int smem = (int)sizeof(cb::ScanSmem<NS, CH>);
+  constexpr int smem = (int)sizeof(cb::ScanSmem<T, NS, CH>);
   static bool granted = false;
   if (!granted && smem > 48 * 1024) {
     if (cudaFuncSetAttribute(cb::selective_scan_kernel<T, NS, CH, FAST>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess)
