@@ -43,6 +43,9 @@ CONFIGS = {
                                                                        mvdim=128, cap=9.0, ff=144),
                   par(heads=2, kv=2, dim=128, scale=0.15, temp=(0.2, 64), mem=3, mdim=128, mvdim=64, cap=15.0, ff=None), scan(of=0, inner=208,
                   state=16, rank=24, conv=4, ff=72)], vocab=200, width=192),
+    # products long enough that a few rows split K: the kernels behind them add up partial sums
+    "wide": config([scan(inner=536, state=12, rank=20, conv=4, ff=528), par(heads=6, kv=2, dim=88, scale=0.1, temp=(0.3, 16), mem=2, mdim=64, mvdim=288,
+                                                                       cap=8.0, ff=544)], vocab=150, width=520),
 }
 
 

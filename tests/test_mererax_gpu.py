@@ -45,19 +45,19 @@ def test_whole_prompt_and_residual_stream(tmp_path, name, dtype):
 
 
 @pytest.mark.parametrize("dtype", [F32, BF16])
-@pytest.mark.parametrize("name,page,n", [("mixed", 5, 61), ("bare", 8, 61), ("chain", 16, 61), ("tc", 8, 150), ("tc", 32, 150)])
+@pytest.mark.parametrize("name,page,n", [("mixed", 5, 61), ("bare", 8, 61), ("chain", 16, 61), ("tc", 8, 150), ("tc", 32, 150), ("wide", 16, 90)])
 def test_portions_equal_the_whole_prompt(tmp_path, name, page, n, dtype):
     checks.portions_and_token_by_token(tmp_path, name, dtype, DEV, TOL[dtype], n=n, page_size=page, fam=FAM)
 
 
 @pytest.mark.parametrize("dtype", [F32, BF16])
-@pytest.mark.parametrize("name", ["mixed", "bare", "tc"])
+@pytest.mark.parametrize("name", ["mixed", "bare", "tc", "wide"])
 def test_batches_of_unequal_requests_equal_each_alone(tmp_path, name, dtype):
     checks.mixed_batches(tmp_path, name, dtype, DEV, TOL[dtype], page_size=16, fam=FAM)
 
 
 @pytest.mark.parametrize("dtype,slack", [(F32, 1e-4), (BF16, 0.2)])
-@pytest.mark.parametrize("name,graph", [("mixed", True), ("tc", True), ("tc", False)])
+@pytest.mark.parametrize("name,graph", [("mixed", True), ("tc", True), ("tc", False), ("wide", True)])
 def test_greedy_generation_through_the_engine(tmp_path, name, graph, dtype, slack):
     checks.greedy_generation(tmp_path, name, dtype, DEV, slack, graph, page_size=8, fam=FAM)
 
