@@ -35,8 +35,11 @@ static_assert(MT_VS == 32, "value rows fill one quarter of the tensor-memory lan
 
 template <int DIM>
 struct MtSmem {
-  static constexpr int KB = DIM / 64;
-  static constexpr int Q = 0, K = KB * MT_TILE, BS = 2 * KB * MT_TILE, VP = BS + KB * MT_BS_BLOCK, VA = VP + MT_TILE, GATES = VA + MT_TILE;
+  static constexpr int KB = DIM / 64, HALVES = DIM > 128 ? 2 : 1, HB = KB / HALVES;   // 64-column blocks; halves of K
+  static constexpr int Q = 0, K = KB * MT_TILE, BS = 2 * KB * MT_TILE, VP = BS + KB * MT_BS_BLOCK, VA = VP + 2 * MT_TILE, GATES = VA + MT_TILE;
+  // the elementwise warps share the state's columns: with 128 columns or more, value rows appear twice (tensor-memory lanes 0 and
+  // 64), so that twice as many warps can reach them
+  static constexpr int PARTS = DIM >= 128 ? 4 : 2, COLS = DIM / PARTS;
   static constexpr int GATE_BUF = (5 * MT_C + 4) * 4;   // a2, M2, c, floor, w | keep
   static constexpr int BAR = GATES + 2 * GATE_BUF;
   static constexpr int USED = BAR + 256 + 1024;
@@ -45,7 +48,8 @@ struct MtSmem {
 static_assert(MtSmem<256>::VP % 1024 == 0 && MtSmem<128>::VP % 1024 == 0 && MtSmem<64>::VP % 1024 == 0 && MtSmem<64>::BAR % 16 == 0 &&
                   MtSmem<256>::BYTES <= 232448, "matrix memory shared memory");
 
-enum : int { MB_QF, MB_KF, MB_QE, MB_KE, MB_GF, MB_GE = MB_GF + 2, MB_XF = MB_GE + 2, MB_SF, MB_PF, MB_OF, MB_COUNT };
+// barriers; K comes and goes in halves of 128 columns (KF, KE), gates in two buffers
+enum : int { MB_QF, MB_QE, MB_KF, MB_KE = MB_KF + 2, MB_GF = MB_KE + 2, MB_GE = MB_GF + 2, MB_XF = MB_GE + 2, MB_SF, MB_PF, MB_OF, MB_COUNT };
 
 __device__ __forceinline__ void mt_ld16(uint32_t taddr, uint32_t (&v)[16]) {
   asm volatile(
@@ -55,6 +59,12 @@ __device__ __forceinline__ void mt_ld16(uint32_t taddr, uint32_t (&v)[16]) {
         "=r"(v[10]), "=r"(v[11]), "=r"(v[12]), "=r"(v[13]), "=r"(v[14]), "=r"(v[15])
       : "r"(taddr)
       : "memory");
+}
+
+// Brings a tile of a tensor map into L2.
+__device__ __forceinline__ void mt_prefetch(const CUtensorMap* m, int x, int y) {
+  asm volatile("cp.async.bulk.prefetch.tensor.2d.L2.global.tile [%0, {%1, %2}];" ::"l"(reinterpret_cast<uint64_t>(m)), "r"(x), "r"(y)
+               : "memory");
 }
 
 // 16-byte piece `chunk` of row `row` in a tile of 128-byte rows with the 128-byte swizzle.
@@ -83,7 +93,7 @@ template <int DIM>
 __global__ void __launch_bounds__(MT_THREADS, 1)
 matrix_memory_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK, const MtParams p) {
   using L = MtSmem<DIM>;
-  constexpr int KB = L::KB;
+  constexpr int KB = L::KB, HB = L::HB, HALVES = L::HALVES;
   extern __shared__ uint8_t smem_raw[];
   const uint32_t base = (smem_u32(smem_raw) + 1023u) & ~1023u;
   uint8_t* gen = smem_raw + (base - smem_u32(smem_raw));
@@ -128,22 +138,38 @@ matrix_memory_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
   if (warp == 8) {
     // ---------------- TMA: Q and K tiles of a chunk
     if (lane == 0) {
-      int issued_q = 0, issued_k = 0;
+      int issued_q = 0, issued_k[HALVES] = {};
+      // a tile is waited for with nothing else to do, so it has to come from L2: the slices of a head share the blocks of the
+      // chunk after the next
+      auto ahead = [&](int j) {
+        if (j >= n_chunks) return;
+        const int x = h * DIM + (slice % KB) * 64, row = pt.row0 + j * MT_C;
+        mt_prefetch(&tmK, x, row);
+        mt_prefetch(&tmQ, x, row);
+      };
+      ahead(1);
       for (int j = 0; j < n_chunks; ++j) {
         const int row = pt.row0 + j * MT_C;
+        ahead(j + 2);
         if (j > 0 && !mbar_wait(B(MB_QE), (j - 1) & 1, abort_flag, p.status, ST_TIMEOUT_TMA)) break;
         mbar_arrive_expect_tx(B(MB_QF), KB * MT_TILE);
         for (int b = 0; b < KB; ++b) tma_load_2d(base + L::Q + b * MT_TILE, &tmQ, B(MB_QF), h * DIM + b * 64, row);
         ++issued_q;
-        if (j > 0 && !mbar_wait(B(MB_KE), (j - 1) & 1, abort_flag, p.status, ST_TIMEOUT_TMA)) break;
-        mbar_arrive_expect_tx(B(MB_KF), KB * MT_TILE);
-        for (int b = 0; b < KB; ++b) tma_load_2d(base + L::K + b * MT_TILE, &tmK, B(MB_KF), h * DIM + b * 64, row);
-        ++issued_k;
+        bool ok = true;
+        for (int f = 0; f < HALVES && ok; ++f) {
+          if (j > 0) ok = mbar_wait(B(MB_KE + f), (j - 1) & 1, abort_flag, p.status, ST_TIMEOUT_TMA);
+          if (!ok) break;
+          mbar_arrive_expect_tx(B(MB_KF + f), HB * MT_TILE);
+          for (int b = f * HB; b < (f + 1) * HB; ++b) tma_load_2d(base + L::K + b * MT_TILE, &tmK, B(MB_KF + f), h * DIM + b * 64, row);
+          ++issued_k[f];
+        }
+        if (!ok) break;
       }
       // copies in flight end before the CTA does, also when a wait gave up
       volatile int no_abort = 0;
       if (issued_q > 0) mbar_wait(B(MB_QF), (issued_q - 1) & 1, &no_abort, nullptr, 0);
-      if (issued_k > 0) mbar_wait(B(MB_KF), (issued_k - 1) & 1, &no_abort, nullptr, 0);
+      for (int f = 0; f < HALVES; ++f)
+        if (issued_k[f] > 0) mbar_wait(B(MB_KF + f), (issued_k[f] - 1) & 1, &no_abort, nullptr, 0);
     }
   } else if (warp == 9) {
     // ---------------- MMA issuer
@@ -151,31 +177,40 @@ matrix_memory_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
       const uint64_t q_desc = make_smem_desc_sw128(base + L::Q, 16, 1024), k_desc = make_smem_desc_sw128(base + L::K, 16, 1024);
       const uint64_t bs_desc = make_smem_desc_sw128(base + L::BS, 16, 1024);
       const uint64_t kt_desc = make_smem_desc_sw128(base + L::K, MT_TILE, 1024);
-      const uint64_t vp_desc = make_smem_desc_sw128(base + L::VP, MT_TILE, 1024);   // value rows 64..127: V itself, never read
+      const uint64_t vp_desc = make_smem_desc_sw128(base + L::VP, MT_TILE, 1024);   // value rows 0..63, and again
       const uint64_t va_desc = make_smem_desc_sw128(base + L::VA, MT_TILE, 1024);
       constexpr uint32_t id_s = make_idesc_bf16(128, 128, 0, 0), id_i = make_idesc_bf16(128, MT_BS_ROWS, 0, 0),
-                         id_u = make_idesc_bf16(128, DIM, 1, 1), id_p = make_idesc_bf16(128, MT_PV_N, 0, 1);
+                         id_u = make_idesc_bf16(128, HB * 64, 1, 1), id_p = make_idesc_bf16(128, MT_PV_N, 0, 1);
       auto wait = [&](int b, int phase) { return mbar_wait(B(b), phase & 1, abort_flag, p.status, ST_TIMEOUT_MMA); };
       for (int j = 0; j < n_chunks; ++j) {
-        if (!wait(MB_QF, j) || !wait(MB_KF, j)) break;
-        tc_fence_after();
-#pragma unroll 1
-        for (int kk = 0; kk < DIM / 16; ++kk) {
-          const uint64_t off = (uint64_t)((kk >> 2) * (MT_TILE >> 4) + 2 * (kk & 3));
-          mma_ss(tmem + MT_T_SCORE, q_desc + off, k_desc + off, id_s, kk > 0);
-        }
-        tc_commit(B(MB_SF));
-        if (!wait(MB_XF, j)) break;
+        // the inter-chunk product first: it needs no K, whose tile is still on its way
+        bool ok = wait(MB_QF, j) && wait(MB_XF, j);
+        if (!ok) break;
         tc_fence_after();
 #pragma unroll 1
         for (int kk = 0; kk < DIM / 16; ++kk)
           mma_ss(tmem + MT_T_INTER, q_desc + (uint64_t)((kk >> 2) * (MT_TILE >> 4) + 2 * (kk & 3)),
                  bs_desc + (uint64_t)((kk >> 2) * (MT_BS_BLOCK >> 4) + 2 * (kk & 3)), id_i, kk > 0);
-        tc_commit(B(MB_QE));
+        for (int f = 0; f < HALVES && ok; ++f) {
+          ok = wait(MB_KF + f, j);
+          if (!ok) break;
+          tc_fence_after();
 #pragma unroll 1
-        for (int kk = 0; kk < MT_C / 16; ++kk)
-          mma_ss(tmem + MT_T_STATE, vp_desc + (uint64_t)(kk * (2048 >> 4)), kt_desc + (uint64_t)(kk * (2048 >> 4)), id_u, 1u);
-        tc_commit(B(MB_KE));
+          for (int kk = f * HB * 4; kk < (f + 1) * HB * 4; ++kk) {
+            const uint64_t off = (uint64_t)((kk >> 2) * (MT_TILE >> 4) + 2 * (kk & 3));
+            mma_ss(tmem + MT_T_SCORE, q_desc + off, k_desc + off, id_s, kk > 0);
+          }
+        }
+        if (!ok) break;
+        tc_commit(B(MB_SF));
+        tc_commit(B(MB_QE));
+        for (int f = 0; f < HALVES; ++f) {
+#pragma unroll 1
+          for (int kk = 0; kk < MT_C / 16; ++kk)
+            mma_ss(tmem + MT_T_STATE + f * HB * 64, vp_desc + (uint64_t)(kk * (2048 >> 4)),
+                   kt_desc + (uint64_t)(f * HB * (MT_TILE >> 4) + kk * (2048 >> 4)), id_u, 1u);
+          tc_commit(B(MB_KE + f));
+        }
         if (!wait(MB_PF, j)) break;
         tc_fence_after();
 #pragma unroll 1
@@ -189,15 +224,42 @@ matrix_memory_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
     const float bi = p.gate_bias[h], bf = p.gate_bias[p.H + h];
     float m_prev = start ? 0.f : *mg;
     bool ok = true;
+    float ni[4], nf[4];   // the next chunk's rows, on their way
+    const float* gp = reinterpret_cast<const float*>(p.gates.p) + h;
+    auto fetch = [&](int j) {
+      const int left = pt.rows - j * MT_C;
+      if (left <= 0) return;
+      const float* r[4];
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        r[e] = gp + (pt.row0 + j * MT_C + min(lane * 4 + e, left - 1)) * p.gates.ld;
+        ni[e] = r[e][0];
+        nf[e] = r[e][p.H];
+      }
+      for (int k = 1; k < p.gates.k_splits; ++k) {
+        float x[8];
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          x[e] = r[e][k * p.gates.split_stride];
+          x[4 + e] = r[e][k * p.gates.split_stride + p.H];
+        }
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          ni[e] += x[e];
+          nf[e] += x[4 + e];
+        }
+      }
+    };
+    fetch(0);
     for (int j = 0; j < n_chunks; ++j) {
       const int cnt = min(MT_C, pt.rows - j * MT_C);
       float gi[4], gf[4];
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
-        const long long row = pt.row0 + j * MT_C + min(lane * 4 + e, cnt - 1);
-        gi[e] = load_source1<float>(p.gates, row, h);
-        gf[e] = load_source1<float>(p.gates, row, p.H + h);
+        gi[e] = ni[e];
+        gf[e] = nf[e];
       }
+      fetch(j + 1);
       float F[4], a[4], sum = 0.f;
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
@@ -273,25 +335,22 @@ matrix_memory_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
       const bool r = mbar_wait(B(b), phase & 1, abort_flag, p.status, ST_TIMEOUT_SOFTMAX);
       return __all_sync(0xffffffffu, r) != 0;
     };
-    fetch_v(0);
-    bool ok = true;
-    for (int j = 0; j < n_chunks; ++j) {
-      const int cnt = min(MT_C, pt.rows - j * MT_C);
-      ok = wait(MB_GF + (j & 1), j >> 1);
-      if (!ok) break;
-      const float* g = gate_buf(j);
-      // ---- the state as operand, then rescaled in place (value rows: quad 0; n: lanes 0 and 1 of quad 1)
-      if (quad < 2) {
-        const float keep = g[5 * MT_C];
+    // The state as operand, then rescaled in place, for chunk j: value rows on even quarters of the lanes, n on lanes 0 and 1 of
+    // odd ones; this warp's columns only.
+    const bool even = (quad & 1) == 0, holds = L::PARTS == 4 || quad < 2;
+    const int col0 = (L::PARTS == 4 ? wg * 2 + (quad >> 1) : wg) * L::COLS;
+    auto convert = [&](int j) {
+      if (holds) {
+        const float keep = gate_buf(j)[5 * MT_C];
 #pragma unroll 1
-        for (int c0 = wg * (DIM / 2); c0 < (wg + 1) * (DIM / 2); c0 += 32) {
+        for (int c0 = col0; c0 < col0 + L::COLS; c0 += 32) {
           uint32_t s[32];
           if (j == 0) {
 #pragma unroll
             for (int i = 0; i < 32; ++i) {
               float x = 0.f;
-              if (!start && quad == 0) x = Sg[(long long)(c0 + i) * p.vdim + lane];
-              if (!start && quad == 1 && lane == 0) x = ng[c0 + i];
+              if (!start && even) x = Sg[(long long)(c0 + i) * p.vdim + lane];
+              if (!start && !even && lane == 0) x = ng[c0 + i];
               s[i] = __float_as_uint(x);
             }
           } else {
@@ -299,8 +358,8 @@ matrix_memory_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
             tmem_wait_ld();
           }
           uint8_t* block = gen + L::BS + (c0 >> 6) * MT_BS_BLOCK;
-          const int row_hi = quad == 0 ? lane : MT_N_COL + 2 * lane;       // n: rows 32 (high), 33 (low), 34 (the low weights' sum)
-          const int row_lo = quad == 0 ? MT_LO + lane : MT_N_COL + 1;
+          const int row_hi = even ? lane : MT_N_COL + 2 * lane;       // n: rows 32 (high), 33 (low), 34 (the low weights' sum)
+          const int row_lo = even ? MT_LO + lane : MT_N_COL + 1;
 #pragma unroll
           for (int q = 0; q < 4; ++q) {
             uint32_t hi[4], lo[4];
@@ -311,8 +370,8 @@ matrix_memory_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
               lo[e] = pack_bf16(x - bf16lo(hi[e]), y - bf16hi(hi[e]));
             }
             const int chunk = ((c0 & 63) >> 3) + q;
-            if (quad == 0 || lane < 2) *mt_piece(block, row_hi, chunk) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
-            if (quad == 0 || lane == 0) *mt_piece(block, row_lo, chunk) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+            if (even || lane < 2) *mt_piece(block, row_hi, chunk) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+            if (even || lane == 0) *mt_piece(block, row_lo, chunk) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
           }
 #pragma unroll
           for (int i = 0; i < 32; ++i) s[i] = __float_as_uint(__uint_as_float(s[i]) * keep);
@@ -320,37 +379,43 @@ matrix_memory_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
           tmem_st32(lane_addr + MT_T_STATE + c0, s);
         }
         tmem_wait_st();
-      } else if (j == 0) {   // value rows 64..127 of the accumulator hold nothing that is used; start them from zero
-        uint32_t z[32];
-#pragma unroll
-        for (int i = 0; i < 32; ++i) z[i] = 0u;
-#pragma unroll 1
-        for (int c0 = wg * (DIM / 2); c0 < (wg + 1) * (DIM / 2); c0 += 32) tmem_st32(lane_addr + MT_T_STATE + c0, z);
-        tmem_wait_st();
       }
-      // ---- V operands: [V | 1] and [w V | w]
-      {
-        const float w = g[4 * MT_C + vt];
-        uint8_t *va = gen + L::VA, *vp = gen + L::VP;
+    };
+    // V operands of chunk j, [V | 1] and [w V | w], then everything that the chunk's products read is in place.
+    auto operands = [&](int j) {
+      const float w = gate_buf(j)[4 * MT_C + vt];
+      uint8_t *va = gen + L::VA, *vp = gen + L::VP, *vp2 = vp + MT_TILE;
 #pragma unroll
-        for (int q = 0; q < 2; ++q) {
-          *mt_piece(va, vt, vh * 2 + q) = vr[q];
-          const uint32_t in[4] = {vr[q].x, vr[q].y, vr[q].z, vr[q].w};
-          uint32_t o[4];
+      for (int q = 0; q < 2; ++q) {
+        *mt_piece(va, vt, vh * 2 + q) = vr[q];
+        const uint32_t in[4] = {vr[q].x, vr[q].y, vr[q].z, vr[q].w};
+        uint32_t o[4];
 #pragma unroll
-          for (int e = 0; e < 4; ++e) o[e] = pack_bf16(w * bf16lo(in[e]), w * bf16hi(in[e]));
-          *mt_piece(vp, vt, vh * 2 + q) = make_uint4(o[0], o[1], o[2], o[3]);
-        }
-        if (vh == 0) {
-          *mt_piece(va, vt, 4) = make_uint4(pack_bf16(vt < cnt ? 1.f : 0.f, 0.f), 0u, 0u, 0u);
-          const float hi = mt_round(w);
-          *mt_piece(vp, vt, 4) = make_uint4(pack_bf16(hi, w - hi), 0u, 0u, 0u);
-        }
+        for (int e = 0; e < 4; ++e) o[e] = pack_bf16(w * bf16lo(in[e]), w * bf16hi(in[e]));
+        *mt_piece(vp, vt, vh * 2 + q) = make_uint4(o[0], o[1], o[2], o[3]);
+        if (L::PARTS == 4) *mt_piece(vp2, vt, vh * 2 + q) = make_uint4(o[0], o[1], o[2], o[3]);
+      }
+      if (vh == 0) {
+        *mt_piece(va, vt, 4) = make_uint4(pack_bf16(j * MT_C + vt < pt.rows ? 1.f : 0.f, 0.f), 0u, 0u, 0u);
+        const float hi = mt_round(w);
+        *mt_piece(vp, vt, 4) = make_uint4(pack_bf16(hi, w - hi), 0u, 0u, 0u);
+        if (L::PARTS == 4) *mt_piece(vp2, vt, 4) = make_uint4(pack_bf16(hi, w - hi), 0u, 0u, 0u);
       }
       fence_proxy_async();
       tc_fence_before();
       mbar_arrive(B(MB_XF));
       if (j + 1 < n_chunks) fetch_v(j + 1);
+    };
+    fetch_v(0);
+    bool ok = wait(MB_GF, 0);
+    if (ok) {
+      convert(0);
+      operands(0);
+    }
+    for (int j = 0; j < n_chunks && ok; ++j) {
+      const int cnt = min(MT_C, pt.rows - j * MT_C);
+      const bool more = j + 1 < n_chunks;
+      const float* g = gate_buf(j);
       // ---- P = scores e^(a_s - M_t), causal; this half's 64 columns in two blocks of 32
       const float M2 = g[MT_C + t], c_t = g[2 * MT_C + t], floor_t = g[3 * MT_C + t];
       ok = wait(MB_SF, j);
@@ -386,6 +451,14 @@ matrix_memory_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
       tmem_wait_st();
       tc_fence_before();
       mbar_arrive(B(MB_PF));
+      mbar_arrive(B(MB_GE + (j & 1)));
+      // ---- the state after this chunk as the next one's operand, beside the last product
+      if (more) {
+        ok = wait(MB_GF + ((j + 1) & 1), (j + 1) >> 1) && wait(MB_KE + HALVES - 1, j);
+        if (!ok) break;
+        tc_fence_after();
+        convert(j + 1);
+      }
       // ---- output: this half's 16 value columns
       ok = wait(MB_OF, j);
       if (!ok) break;
@@ -397,8 +470,7 @@ matrix_memory_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
       mt_ld16(lane_addr + MT_T_INTRA + wg * 16, in);
       mt_ld16(lane_addr + MT_T_INTRA + MT_N_COL, ni);
       tmem_wait_ld();
-      tc_fence_before();
-      mbar_arrive(B(MB_GE + (j & 1)));
+      if (more) operands(j + 1);
       auto f = [](uint32_t u) { return __uint_as_float(u); };
       const float nq = fmaf(c_t, f(nn[0]) + (f(nn[1]) + f(nn[2])), f(ni[0]));
       const float inv = 1.f / (fmaxf(fabsf(nq), floor_t) + 1e-6f);
@@ -415,17 +487,17 @@ matrix_memory_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
       __syncwarp();
     }
     // ---- the state back to memory
-    if (ok && quad < 2) {
+    if (ok && holds) {
 #pragma unroll 1
-      for (int c0 = wg * (DIM / 2); c0 < (wg + 1) * (DIM / 2); c0 += 32) {
+      for (int c0 = col0; c0 < col0 + L::COLS; c0 += 32) {
         uint32_t s[32];
         tmem_ld32(lane_addr + MT_T_STATE + c0, s);
         tmem_wait_ld();
 #pragma unroll
         for (int i = 0; i < 32; ++i) {
           const float x = __uint_as_float(s[i]), other = __shfl_down_sync(0xffffffffu, x, 1);
-          if (quad == 0) Sg[(long long)(c0 + i) * p.vdim + lane] = x;
-          if (quad == 1 && lane == 0) ng[c0 + i] = x + other;
+          if (even) Sg[(long long)(c0 + i) * p.vdim + lane] = x;
+          if (!even && lane == 0) ng[c0 + i] = x + other;
         }
         __syncwarp();
       }
