@@ -172,7 +172,7 @@ matrix_memory_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
         if (issued_k[f] > 0) mbar_wait(B(MB_KF + f), (issued_k[f] - 1) & 1, &no_abort, nullptr, 0);
     }
   } else if (warp == 9) {
-    // ---------------- MMA issuer
+    // ---------------- MMA issuer (unrolled: descriptor arithmetic between two products would cost more than a product)
     if (lane == 0) {
       const uint64_t q_desc = make_smem_desc_sw128(base + L::Q, 16, 1024), k_desc = make_smem_desc_sw128(base + L::K, 16, 1024);
       const uint64_t bs_desc = make_smem_desc_sw128(base + L::BS, 16, 1024);
@@ -187,15 +187,16 @@ matrix_memory_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
         bool ok = wait(MB_QF, j) && wait(MB_XF, j);
         if (!ok) break;
         tc_fence_after();
-#pragma unroll 1
+#pragma unroll
         for (int kk = 0; kk < DIM / 16; ++kk)
           mma_ss(tmem + MT_T_INTER, q_desc + (uint64_t)((kk >> 2) * (MT_TILE >> 4) + 2 * (kk & 3)),
                  bs_desc + (uint64_t)((kk >> 2) * (MT_BS_BLOCK >> 4) + 2 * (kk & 3)), id_i, kk > 0);
-        for (int f = 0; f < HALVES && ok; ++f) {
-          ok = wait(MB_KF + f, j);
+#pragma unroll
+        for (int f = 0; f < HALVES; ++f) {
+          ok = ok && wait(MB_KF + f, j);
           if (!ok) break;
           tc_fence_after();
-#pragma unroll 1
+#pragma unroll
           for (int kk = f * HB * 4; kk < (f + 1) * HB * 4; ++kk) {
             const uint64_t off = (uint64_t)((kk >> 2) * (MT_TILE >> 4) + 2 * (kk & 3));
             mma_ss(tmem + MT_T_SCORE, q_desc + off, k_desc + off, id_s, kk > 0);
@@ -204,8 +205,9 @@ matrix_memory_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
         if (!ok) break;
         tc_commit(B(MB_SF));
         tc_commit(B(MB_QE));
+#pragma unroll
         for (int f = 0; f < HALVES; ++f) {
-#pragma unroll 1
+#pragma unroll
           for (int kk = 0; kk < MT_C / 16; ++kk)
             mma_ss(tmem + MT_T_STATE + f * HB * 64, vp_desc + (uint64_t)(kk * (2048 >> 4)),
                    kt_desc + (uint64_t)(f * HB * (MT_TILE >> 4) + kk * (2048 >> 4)), id_u, 1u);
@@ -213,7 +215,7 @@ matrix_memory_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_co
         }
         if (!wait(MB_PF, j)) break;
         tc_fence_after();
-#pragma unroll 1
+#pragma unroll
         for (int kk = 0; kk < MT_C / 16; ++kk)
           mma_ts(tmem + MT_T_INTRA, tmem + MT_T_SCORE + (kk >> 2) * 64 + (kk & 3) * 8, va_desc + (uint64_t)(kk * (2048 >> 4)), id_p, kk > 0);
         tc_commit(B(MB_OF));
