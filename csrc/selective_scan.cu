@@ -49,10 +49,13 @@ causal_conv_rows_kernel(const cosmos::CausalConvArgs a) {
     }
   }
   Vec<float, 8>::load(a.b + c, bias);
+  float wr[8 * TAPS];   // the 8 channels' taps lie side by side
+#pragma unroll
+  for (int k = 0; k < 2 * TAPS; ++k) Vec<float, 4>::load(a.w + (long long)c * TAPS + 4 * k, *reinterpret_cast<float(*)[4]>(&wr[4 * k]));
 #pragma unroll
   for (int e = 0; e < 8; ++e)
 #pragma unroll
-    for (int j = 0; j < TAPS; ++j) w[j][e] = a.w[(long long)(c + e) * TAPS + j];
+    for (int j = 0; j < TAPS; ++j) w[j][e] = wr[e * TAPS + j];
   for (int r8 = 0; r8 < rows; r8 += AHEAD) {
 #pragma unroll
     for (int i = 0; i < AHEAD; ++i) {
@@ -565,7 +568,7 @@ template <typename T>
 static void launch_conv(const CausalConvArgs& a, cudaStream_t s) {
   auto on = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
   const bool vec = a.inner % 8 == 0 && a.x.ld % 8 == 0 && a.x.split_stride % 8 == 0 && a.ldu % 8 == 0 && on(a.x.p) && on(a.u) &&
-                   on(a.conv_state) && on(a.b);
+                   on(a.conv_state) && on(a.b) && on(a.w);
   const int v = vec && a.taps <= 4 ? 8 : 1;
   const int per = (a.inner + v - 1) / v, threads = std::min(128, (per + 31) / 32 * 32);
   const dim3 grid((per + threads - 1) / threads, a.tiles ? a.n_tiles : a.rows.n);

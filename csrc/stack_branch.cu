@@ -128,6 +128,7 @@ qk_norm_post_kernel(const cosmos::QkNormArgs a) {
   const long long r = blockIdx.x;
   const int tid = threadIdx.x, nt = blockDim.x;
   const int qc = a.H * a.dim, kc = a.G * a.dim;
+  const long long slot = a.slots[r], pos = a.temp_every > 0 ? a.positions[r] : 0;
   float q[NV][VEC], k[NV][VEC];
   float sq = 0.f, sk = 0.f;
 #pragma unroll
@@ -148,10 +149,9 @@ qk_norm_post_kernel(const cosmos::QkNormArgs a) {
   float rq = 1.f / sqrtf(ss.x / (float)qc + a.eps);
   const float rk = 1.f / sqrtf(ss.y / (float)kc + a.eps);
   if (a.temp_every > 0) {
-    const unsigned step = (unsigned)(a.positions[r] + 1) / (unsigned)a.temp_every;   // positions fit 32 bits
+    const unsigned step = (unsigned)(pos + 1) / (unsigned)a.temp_every;   // positions fit 32 bits
     rq *= 1.f + a.temp_coef * logf((float)(step + 1));
   }
-  const long long slot = a.slots[r];
   const bool ok = index_ok(slot, a.n_slots, a.status, SITE_STACK_SLOT);
   const unsigned page = ok ? (unsigned)slot / (unsigned)a.page_size : 0u;
   const int off = ok ? (int)((unsigned)slot - page * (unsigned)a.page_size) : 0;
@@ -229,7 +229,9 @@ static void launch_qk(const QkNormArgs& a, cudaStream_t s) {
   const bool vec = a.dim % 8 == 0 && vec8_source(a.q) && vec8_source(a.k) && on(a.wq, 16) && on(a.wk, 16) && on(a.q_out, 16) &&
                    on(a.k_cache, 16) && on(a.v_cache, 16);
   const unsigned rows = (unsigned)a.n;
-  if (vec && cols <= 8192)
+  if (vec && cols <= 8192 && cols > 1024 && a.n > 296)
+    cb::qk_norm_post_kernel<T, 8, 2, PART><<<rows, row_threads(cols, 8, 2), 0, s>>>(a);
+  else if (vec && cols <= 8192)
     cb::qk_norm_post_kernel<T, 8, 1, PART><<<rows, row_threads(cols, 8, 1), 0, s>>>(a);
   else if (cols <= 1024)
     cb::qk_norm_post_kernel<T, 1, 1, PART><<<rows, row_threads(cols, 1, 1), 0, s>>>(a);
