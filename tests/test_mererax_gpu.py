@@ -274,7 +274,7 @@ def test_selective_scan_and_its_state(dtype, inner, ns, partial):
             assert float(y[:, inner:c8].float().abs().sum()) == 0 and float((y[:, c8:] - 7).float().abs().max()) == 0
 
 
-MEMORIES = [(3, 10, 22, 7.0), (2, 32, 64, 12.0), (1, 16, 9, 3.0), (2, 64, 128, 9.0), (1, 128, 64, 15.0), (2, 256, 96, 12.0), (1, 3, 33, 5.0), (1, 300, 40, 6.0),
+MEMORIES = [(3, 10, 22, 7.0), (2, 40, 64, 11.0), (1, 16, 9, 3.0), (2, 64, 128, 9.0), (1, 128, 64, 15.0), (2, 256, 96, 12.0), (1, 3, 33, 5.0), (1, 300, 40, 6.0),
             (2, 128, 192, 4.0)]
 
 
